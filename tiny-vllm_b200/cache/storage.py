@@ -5,8 +5,9 @@ head_dim]`` (keys, and values, whose last size may differ) in the storage dtype:
 page are contiguous, so a kernel that serves one kv head reads whole runs of
 memory.  Token ``p`` of a request lies in page ``block_table[p // page_size]``
 at offset ``p % page_size`` of every run of the group (its *slot* is
-``page * page_size + offset``).  A run that declares fixed-size state owns an arena
-``[state_slots, *shape]``; a request's row is zeroed when the request starts.
+``page * page_size + offset``).  A run that declares fixed-size states owns an arena
+``[state_slots, *shape]`` for each, beside its pages if it keeps keys and values too; a request's
+row is zeroed when the request starts.  So does an embedding that carries something from token to token.
 The reference keeps one pair of tensors ``[layers, blocks * block_size,
 kv_heads, head_dim]`` (tinyvllm/paged_kv.py:53-65).
 """
@@ -15,7 +16,7 @@ from __future__ import annotations
 
 import torch
 
-from ..parts.base import KVNeed, StateNeed
+from ..parts.base import kv_need, state_needs
 from .manager import CacheGroup
 
 
@@ -26,8 +27,9 @@ def group_runs(needs: list, cache_from: list) -> tuple[list[CacheGroup], dict[in
     geometries: list[tuple] = []
     members: list[list[int]] = []
     where: dict[int, tuple[int, int]] = {}
+    needs = [kv_need(need) for need in needs]
     for run, need in enumerate(needs):
-        if not isinstance(need, KVNeed) or cache_from[run] is not None:
+        if need is None or cache_from[run] is not None:
             continue
         for g, geometry in enumerate(geometries):
             if geometry == need.geometry():
@@ -47,7 +49,7 @@ def group_runs(needs: list, cache_from: list) -> tuple[list[CacheGroup], dict[in
         if source is None:
             continue
         need, theirs = needs[run], needs[source]
-        if not isinstance(need, KVNeed) or not isinstance(theirs, KVNeed) or (
+        if need is None or theirs is None or (
                 need.num_kv_heads, need.head_dim, need.value_size) != (
                     theirs.num_kv_heads, theirs.head_dim, theirs.value_size):
             raise ValueError(f"run {run} cannot read the cache of run {source}: shapes differ")
@@ -64,7 +66,7 @@ def bytes_per_page(group: CacheGroup, page_size: int, itemsize: int) -> int:
 
 class CacheStorage:
     def __init__(self, groups, where, needs, *, page_size: int, pages_per_group,
-                 num_state_slots: int, dtype: torch.dtype, device) -> None:
+                 num_state_slots: int, dtype: torch.dtype, device, other_states: dict | None = None) -> None:
         self.groups = tuple(groups)
         self.where = dict(where)
         self.page_size = page_size
@@ -83,11 +85,12 @@ class CacheStorage:
                 if not 0 <= group.value_offset <= group.head_dim - group.value_size:
                     raise ValueError("values inside the key rows must fit them")
                 self.values.append(None)
-        self.state: dict[int, torch.Tensor] = {}
-        for run, need in enumerate(needs):
-            if isinstance(need, StateNeed):
-                self.state[run] = torch.zeros(
-                    (num_state_slots,) + tuple(need.shape), dtype=need.dtype, device=device)
+        # run -> arena, (run, name) -> arena for states with names; ``other_states`` are those of no run
+        self.state: dict = {}
+        for key, need in [*enumerate(needs), *(other_states or {}).items()]:
+            for state in state_needs(need):
+                self.state[(key, state.name) if state.name else key] = torch.zeros(
+                    (num_state_slots,) + tuple(state.shape), dtype=state.dtype, device=device)
 
     def group_of(self, run: int) -> int:
         return self.where[run][0]
@@ -98,8 +101,9 @@ class CacheStorage:
         values = self.values[group]
         return self.keys[group][index], None if values is None else values[index]
 
-    def state_of(self, run: int) -> torch.Tensor:
-        return self.state[run]
+    def state_of(self, run, name: str = "") -> torch.Tensor:
+        """The arena of a run's state (of the state called ``name``, for a run with several)."""
+        return self.state[(run, name) if name else run]
 
     def clear_state(self, slots) -> None:
         """Zero the state rows of requests that start in this step."""

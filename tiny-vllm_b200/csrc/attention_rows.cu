@@ -93,10 +93,12 @@ __device__ __forceinline__ float dot_head<bf16>(const float* __restrict__ q_shar
     return dot;
 }
 
-// What is added to a score beside the scaled product: `slope` > 0 takes slope * (position - j) off the
+// What becomes of a score beside the scaled product: `softcap` > 0 first turns it into softcap * tanh(score /
+// softcap); `slope` > 0 takes slope * (position - j) off the
 // score of key j; `table` (or null) holds one learned number a distance, `stride` floats apart, and
 // table[min(position - j, rows - 1) * stride] is added (all distances from rows - 1 on share the last).
 struct ScoreBias {
+    float softcap;
     float slope;
     const float* table;
     int rows;
@@ -132,6 +134,7 @@ __device__ __forceinline__ void attend_chunk(
             slot = ((int64_t)table[j / page_size] * num_kv + kv_head) * page_size + j % page_size;
             const T* k = key_cache + slot * head_dim;
             score = __fmul_rn(dot_head<T>(q_shared, k, head_dim), scale);
+            if (bias.softcap > 0.0f) score = __fmul_rn(bias.softcap, tanhf(__fdiv_rn(score, bias.softcap)));
             if (bias.slope != 0.0f) score = __fsub_rn(score, __fmul_rn(bias.slope, (float)(position - j)));
             if (bias.table) score = __fadd_rn(score, bias.table[(int64_t)min(position - j, bias.rows - 1) * bias.stride]);
         }
@@ -203,6 +206,7 @@ struct RowExtras {
     const float* bias_table;      // float32 [bias_rows, num_q] (or null): a learned number a distance and head
     int bias_rows;
     int segment;                  // > 0: a query sees only the keys of its own segment of so many positions
+    float softcap;                // > 0: scores are capped by softcap * tanh(score / softcap)
 };
 
 // (M, L, O) of a finished row -> output: the sink joins the denominator, then division, gate, rounding.
@@ -265,7 +269,7 @@ __global__ void paged_attention_rows_kernel(
     __syncwarp();
     const int* table = block_tables + (int64_t)request * table_stride;
     const int kv_head = head / (num_q / num_kv);
-    const ScoreBias bias{extras.slopes ? extras.slopes[head] : 0.0f,
+    const ScoreBias bias{extras.softcap, extras.slopes ? extras.slopes[head] : 0.0f,
                          extras.bias_table ? extras.bias_table + head : nullptr, extras.bias_rows, num_q};
 
     if (SPLIT) {
@@ -389,7 +393,8 @@ static void launch_rows(const void* q, long long q_token_stride, const void* key
 // the denominator (`sinks`), and values that lie `value_stride` elements apart (0: value_dim), which
 // lets them be a part of the key rows.
 // `bias_table` (float32 [bias_rows, num_q], or null): table[min(p - j, bias_rows - 1), h] is added to the
-// score of key j; `segment` > 0: the query at p sees only keys from p - p % segment on.
+// score of key j; `segment` > 0: the query at p sees only keys from p - p % segment on; `softcap` > 0: a scaled
+// score s becomes softcap * tanh(s / softcap).
 extern "C" int tvb_attention_rows_masked(const void* q, long long q_token_stride, const void* key_cache,
                                          const void* value_cache, long long value_stride, const int* block_tables,
                                          int table_stride, const int* token_row, const int* positions, void* out,
@@ -398,7 +403,7 @@ extern "C" int tvb_attention_rows_masked(const void* q, long long q_token_stride
                                          const float* bias_table, int bias_rows, int segment,
                                          float* scratch, int max_chunks, int tokens, int num_q, int num_kv,
                                          int head_dim, int value_dim, int page_size, int window, int keep_first,
-                                         float scale, int dtype, void* stream) {
+                                         float scale, float softcap, int dtype, void* stream) {
     if (tokens <= 0) return 0;
     if (segment < 0 || (bias_table && bias_rows <= 0)) return TVB_BAD_ARGUMENT;
     if (head_dim <= 0 || head_dim > 32 * ATTN_WIDE_DIMS || value_dim <= 0 || value_dim > 32 * ATTN_WIDE_DIMS ||
@@ -411,7 +416,7 @@ extern "C" int tvb_attention_rows_masked(const void* q, long long q_token_stride
     if (blocks > 2147483647LL) return TVB_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     RowExtras extras{slopes, sinks, gate_per_head, value_stride > 0 ? value_stride : value_dim,
-                     bias_table, bias_rows, segment};
+                     bias_table, bias_rows, segment, softcap};
     const bool wide = head_dim > 32 * ATTN_MAX_DIMS || value_dim > 32 * ATTN_MAX_DIMS;
 #define LAUNCH_ROWS(T, DIMS)                                                                             \
     launch_rows<T, DIMS>(q, q_token_stride, key_cache, value_cache, block_tables, table_stride, token_row, \
@@ -437,7 +442,7 @@ extern "C" int tvb_attention_rows_biased(const void* q, long long q_token_stride
                                      table_stride, token_row, positions, out, out_token_stride, gate,
                                      gate_token_stride, gate_per_head, slopes, sinks, nullptr, 0, 0, scratch,
                                      max_chunks, tokens, num_q, num_kv, head_dim, value_dim, page_size, window,
-                                     keep_first, scale, dtype, stream);
+                                     keep_first, scale, 0.0f, dtype, stream);
 }
 
 extern "C" int tvb_attention_rows_general(const void* q, long long q_token_stride, const void* key_cache,

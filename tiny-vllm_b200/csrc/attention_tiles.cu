@@ -5,7 +5,8 @@
 // a value, or one a head), an optional distance bias (head h takes slopes[h] * (p - j) off the score of
 // key j) and an optional sink a head (exp(sink) is added to the softmax's denominator and to nothing
 // else), an optional learned bias by distance (bias_table[min(p - j, rows - 1), h] is added to the scaled
-// score) and optional segments (a query sees only the keys from the start of its own segment of
+// score), an optional cap on the scaled scores (s becomes softcap * tanh(s / softcap), before any bias) and
+// optional segments (a query sees only the keys from the start of its own segment of
 // `segment` positions, counted from position 0; not together with a window).  Compiled with TILES_VALUE_IN_KEY=1 the values are the first TILES_VALUE_DIM elements of the
 // key rows themselves (attention over latents that serve as keys and values): no value cache is read
 // and the key tile in shared memory is the value tile too.
@@ -87,6 +88,7 @@ struct TileArgs {
     float scale;
     const float* slopes; const float* sinks; int gate_per_head;
     const float* bias_table; int bias_rows; int segment;
+    float softcap;
 };
 
 // The first key the query at `position` sees (kept first keys apart): the start of its segment of
@@ -102,6 +104,17 @@ __device__ __forceinline__ float table_bias(const TileArgs& a, int distance, int
 }
 
 __device__ __forceinline__ int chunk_of_slot(int z, int window_chunks, int position, int lo, int kept);
+
+// cap * tanh(s / cap) for a score in units of log 2: tanh(x) = 1 - 2 / (1 + e^2x), off by a few units in the last
+// place of 1 at most and clean at both ends
+struct ScoreCap {
+    float cap, inverse;
+    __device__ __forceinline__ ScoreCap(float softcap)
+        : cap(softcap * TL_LOG2E), inverse(softcap > 0.0f ? 2.0f / softcap : 0.0f) {}
+    __device__ __forceinline__ float operator()(float s) const {
+        return cap - __fdividef(2.0f * cap, 1.0f + exp2f(s * inverse));
+    }
+};
 
 template <int KD, int VD, bool SINGLES>
 __global__ void __launch_bounds__(TL_WARPS * 32, 3) attention_tiles_kernel(const TileArgs a) {
@@ -236,6 +249,8 @@ __global__ void __launch_bounds__(TL_WARPS * 32, 3) attention_tiles_kernel(const
     const float slope_a = biased ? a.slopes[head_a] * TL_LOG2E : 0.0f;
     const float slope_b = biased ? a.slopes[head_b] * TL_LOG2E : 0.0f;
     const bool tabled = a.bias_table != nullptr;
+    const bool capped = a.softcap > 0.0f;
+    const ScoreCap cap(a.softcap);
 
     for (int t = 0; t < tiles; ++t) {
         const int buffer = t & 1;
@@ -283,6 +298,7 @@ __global__ void __launch_bounds__(TL_WARPS * 32, 3) attention_tiles_kernel(const
                 const int key = key0 + n * 8 + 2 * t4 + (i & 1);
                 const bool upper = i < 2;
                 float s = s_acc[n][i] * scale_log2;
+                if (capped) s = cap(s);
                 if (biased) s -= (upper ? slope_a : slope_b) * (float)((upper ? pos_a : pos_b) - key);
                 if (tabled) s += table_bias(a, (upper ? pos_a : pos_b) - key, upper ? head_a : head_b);
                 if (!full) {
@@ -516,7 +532,8 @@ __global__ void __launch_bounds__(TL_WARPS * 32, 3) attention_singles_kernel(con
             }
         }
         const float scale_log2 = a.scale * TL_LOG2E;
-        const bool biased = a.slopes != nullptr;
+        const bool biased = a.slopes != nullptr, capped = a.softcap > 0.0f;
+        const ScoreCap cap(a.softcap);
         const float slope_a = biased ? a.slopes[head0 + min(g, group - 1)] * TL_LOG2E : 0.0f;
         const float slope_b = biased ? a.slopes[head0 + min(g + 8, group - 1)] * TL_LOG2E : 0.0f;
 #pragma unroll
@@ -525,6 +542,7 @@ __global__ void __launch_bounds__(TL_WARPS * 32, 3) attention_singles_kernel(con
             for (int i = 0; i < 4; ++i) {
                 const int key = tile_key + n * 8 + 2 * t4 + (i & 1);
                 float s = s_acc[n][i] * scale_log2;
+                if (capped) s = cap(s);
                 if (biased) s -= (i < 2 ? slope_a : slope_b) * (float)(position - key);
                 if (a.bias_table) s += table_bias(a, position - key, head0 + min(i < 2 ? g : g + 8, group - 1));
                 if (!(key <= position && (key >= lo || key < kept))) s = -INFINITY;
@@ -694,7 +712,7 @@ static size_t tiles_shared_bytes() {
 }
 
 static int check_common(const TileArgs& a, int key_dim, int value_dim) {
-    if (a.segment < 0 || (a.segment > 0 && a.window > 0) || (a.bias_table && a.bias_rows <= 0)) return TVB_BAD_ARGUMENT;
+    if (!(a.softcap >= 0.0f) || a.segment < 0 || (a.segment > 0 && a.window > 0) || (a.bias_table && a.bias_rows <= 0)) return TVB_BAD_ARGUMENT;
     if (key_dim != TILES_KEY_DIM || value_dim != TILES_VALUE_DIM || TILES_KEY_DIM % 16 || TILES_VALUE_DIM % 16 ||
         a.num_q <= 0 || a.num_kv <= 0 || a.num_q % a.num_kv || a.page_size <= 0 || a.window < 0 || a.keep_first < 0 ||
         (a.q_token_stride * 2) % 16 || ((uintptr_t)a.q) % 16 || a.out_token_stride % 2 || ((uintptr_t)a.out) % 4 ||
@@ -707,7 +725,7 @@ static int check_common(const TileArgs& a, int key_dim, int value_dim) {
 // Prompt portions: tile i holds tile_count[i] (1..64) consecutive tokens from flat index tile_first[i]
 // on, of the request in row tile_row[i] of block_tables.
 // `slopes` and `sinks`: float32 [num_q] or null; `gate_per_head`: the gate holds one number a head.
-// `bias_table`: float32 [bias_rows, num_q] or null; `segment`: 0 for none.
+// `bias_table`: float32 [bias_rows, num_q] or null; `segment`: 0 for none; `softcap`: 0 for none.
 extern "C" int tvb_attention_tiles_table(const void* q, long long q_token_stride, const void* key_cache,
                                          const void* value_cache, const int* block_tables, int table_stride,
                                          const int* positions, const int* tile_row, const int* tile_first,
@@ -716,12 +734,12 @@ extern "C" int tvb_attention_tiles_table(const void* q, long long q_token_stride
                                          const float* slopes, const float* sinks, const float* bias_table,
                                          int bias_rows, int segment, int tiles, int num_q, int num_kv,
                                          int key_dim, int value_dim, int page_size, int window, int keep_first,
-                                         float scale, void* stream) {
+                                         float scale, float softcap, void* stream) {
     if (tiles <= 0) return 0;
     TileArgs a{(const bf16*)q, q_token_stride, (const bf16*)key_cache, (const bf16*)value_cache, block_tables,
                table_stride, positions, nullptr, tile_row, tile_first, tile_count, (bf16*)out, out_token_stride,
                (const bf16*)gate, gate_token_stride, nullptr, 0, 0, num_q, num_kv, page_size, window,
-               window > 0 ? keep_first : 0, scale, slopes, sinks, gate_per_head, bias_table, bias_rows, segment};
+               window > 0 ? keep_first : 0, scale, slopes, sinks, gate_per_head, bias_table, bias_rows, segment, softcap};
     if (check_common(a, key_dim, value_dim) || num_q > 65535) return TVB_BAD_ARGUMENT;
     auto kernel = attention_tiles_kernel<TILES_KEY_DIM, TILES_VALUE_DIM, false>;
     const size_t shared = tiles_shared_bytes();
@@ -742,7 +760,7 @@ extern "C" int tvb_attention_tiles_biased(const void* q, long long q_token_strid
     return tvb_attention_tiles_table(q, q_token_stride, key_cache, value_cache, block_tables, table_stride, positions,
                                      tile_row, tile_first, tile_count, out, out_token_stride, gate, gate_token_stride,
                                      gate_per_head, slopes, sinks, nullptr, 0, 0, tiles, num_q, num_kv, key_dim,
-                                     value_dim, page_size, window, keep_first, scale, stream);
+                                     value_dim, page_size, window, keep_first, scale, 0.0f, stream);
 }
 
 extern "C" int tvb_attention_tiles(const void* q, long long q_token_stride, const void* key_cache,
@@ -785,12 +803,13 @@ extern "C" int tvb_attention_tiles_singles_table(const void* q, long long q_toke
                                                  const float* sinks, const float* bias_table, int bias_rows,
                                                  int segment, float* scratch, int tokens, int num_q,
                                                  int num_kv, int key_dim, int value_dim, int page_size, int window,
-                                                 int keep_first, float scale, int max_context, void* stream) {
+                                                 int keep_first, float scale, float softcap, int max_context,
+                                                 void* stream) {
     if (tokens <= 0) return 0;
     TileArgs a{(const bf16*)q, q_token_stride, (const bf16*)key_cache, (const bf16*)value_cache, block_tables,
                table_stride, positions, token_row, nullptr, nullptr, nullptr, (bf16*)out, out_token_stride,
                (const bf16*)gate, gate_token_stride, scratch, 0, 0, num_q, num_kv, page_size, window,
-               window > 0 ? keep_first : 0, scale, slopes, sinks, gate_per_head, bias_table, bias_rows, segment};
+               window > 0 ? keep_first : 0, scale, slopes, sinks, gate_per_head, bias_table, bias_rows, segment, softcap};
     if (check_common(a, key_dim, value_dim) || !scratch || max_context <= 0 || num_q / num_kv > TL_BM || num_kv > 65535)
         return TVB_BAD_ARGUMENT;
     singles_chunks(a.segment > 0 ? a.segment : a.window, a.keep_first, max_context, &a.window_chunks, &a.kept_chunks);
@@ -828,7 +847,7 @@ extern "C" int tvb_attention_tiles_singles_biased(const void* q, long long q_tok
     return tvb_attention_tiles_singles_table(q, q_token_stride, key_cache, value_cache, block_tables, table_stride,
                                              positions, token_row, out, out_token_stride, gate, gate_token_stride,
                                              gate_per_head, slopes, sinks, nullptr, 0, 0, scratch, tokens, num_q,
-                                             num_kv, key_dim, value_dim, page_size, window, keep_first, scale,
+                                             num_kv, key_dim, value_dim, page_size, window, keep_first, scale, 0.0f,
                                              max_context, stream);
 }
 

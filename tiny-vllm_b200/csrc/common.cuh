@@ -84,6 +84,31 @@ __device__ __forceinline__ uint4 pack_bf16x8(const float* f) {
                       pack_bf16x2(f[6], f[7]));
 }
 
+// ---- VEC neighbouring values in one access (4: 16 bytes of float32, 8 of bfloat16; 1: a plain access)
+template <int VEC> __device__ __forceinline__ void load_values(const float* p, float* v) {
+    static_assert(VEC == 1 || VEC == 4, "load_values");
+    if constexpr (VEC == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+    } else v[0] = *p;
+}
+template <int VEC> __device__ __forceinline__ void load_values(const bf16* p, float* v) {
+    static_assert(VEC == 1 || VEC == 4, "load_values");
+    if constexpr (VEC == 4) {
+        const uint2 x = *reinterpret_cast<const uint2*>(p);
+        v[0] = __uint_as_float(x.x << 16); v[1] = __uint_as_float(x.x & 0xffff0000u);
+        v[2] = __uint_as_float(x.y << 16); v[3] = __uint_as_float(x.y & 0xffff0000u);
+    } else v[0] = __bfloat162float(*p);
+}
+template <int VEC> __device__ __forceinline__ void store_values(float* p, const float* v) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+}
+template <int VEC> __device__ __forceinline__ void store_values(bf16* p, const float* v) {
+    if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+    else *p = __float2bfloat16_rn(v[0]);
+}
+
 // ---- the cluster's barrier in two halves: arrive early, wait where the others are needed
 __device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory"); }
 // The same without ordering any memory access: for "this CTA runs", said at a kernel's start, where

@@ -36,6 +36,72 @@ extern "C" int tvb_embed_rows(const void* table, const int* ids, void* out, int 
     return tvb_last_error();
 }
 
+// out[t] = table[ids[t]] + pairs[(prev * mul_prev + ids[t] * mul_cur) mod buckets] in float32, prev being the
+// token before t in its request: the step's own, or, for the first token of an entry, the one `state`
+// [slots] keeps from the step before.  A request's first token (position 0) reads the last row, number
+// `buckets`.  The block of an entry's first token is also the one that leaves the entry's last token in the
+// state, so that no block reads what another writes.  `pairs` null: only the table's rows.
+template <typename T, int VEC>
+__global__ void embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs,
+                                   const int* __restrict__ ids, const int* __restrict__ positions,
+                                   const int* __restrict__ token_row, const int* __restrict__ row_starts,
+                                   const int* __restrict__ state_slots, int* state, float* __restrict__ out,
+                                   int width, int vocab, int buckets, int mul_prev, int mul_cur) {
+    const int token = blockIdx.x;
+    int id = ids[token];
+    if (id < 0 || id >= vocab) id = 0;   // the host validates ids; padding rows carry 0
+    const T* src = table + (int64_t)id * width;
+    const T* more = nullptr;
+    const int row = token_row[token];
+    if (pairs && row >= 0) {
+        const int first = row_starts[row], slot = state_slots[row];
+        int bucket = buckets;
+        if (positions[token] > 0) {
+            const int64_t previous = token > first ? ids[token - 1] : state[slot];
+            bucket = (int)((previous * mul_prev + (int64_t)id * mul_cur) % buckets);
+            if (bucket < 0 || bucket >= buckets) bucket = 0;
+        }
+        more = pairs + (int64_t)bucket * width;
+        if (token == first) {
+            __syncthreads();             // every thread of the block has read the state
+            if (threadIdx.x == 0) state[slot] = ids[row_starts[row + 1] - 1];
+        }
+    }
+    float* dst = out + (int64_t)token * width;
+    for (int i = threadIdx.x * VEC; i < width; i += blockDim.x * VEC) {
+        float a[VEC], b[VEC];
+        load_values<VEC>(src + i, a);
+        if (more) {
+            load_values<VEC>(more + i, b);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) a[j] = __fadd_rn(a[j], b[j]);
+        }
+        store_values<VEC>(dst + i, a);
+    }
+}
+
+extern "C" int tvb_embed_pairs(const void* table, const void* pairs, const int* ids, const int* positions,
+                               const int* token_row, const int* row_starts, const int* state_slots, int* state,
+                               float* out, int tokens, int width, int vocab, int buckets, int mul_prev, int mul_cur,
+                               int dtype, void* stream) {
+    if (tokens <= 0) return 0;
+    if (width <= 0 || vocab <= 0 || (pairs && (buckets <= 0 || !state))) return TVB_BAD_ARGUMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t element = dtype == TVB_BF16 ? 2 : 4;
+    const bool by_four = width % 4 == 0 && (uintptr_t)table % (4 * element) == 0 && (uintptr_t)pairs % (4 * element) == 0 &&
+                         (uintptr_t)out % 16 == 0;
+    const int per = by_four ? width / 4 : width;
+    const int threads = per >= 512 ? 256 : (per >= 128 ? 128 : 64);
+#define GO(T, VEC) embed_pairs_kernel<T, VEC><<<tokens, threads, 0, s>>>(                                              \
+        (const T*)table, (const T*)pairs, ids, positions, token_row, row_starts, state_slots, state, out, width, vocab, \
+        buckets, mul_prev, mul_cur)
+    if (dtype == TVB_F32) { if (by_four) GO(float, 4); else GO(float, 1); }
+    else if (dtype == TVB_BF16) { if (by_four) GO(bf16, 4); else GO(bf16, 1); }
+    else return TVB_BAD_ARGUMENT;
+#undef GO
+    return tvb_last_error();
+}
+
 // -------------------------------------------------------------------- RMSNorm
 // One block per output row.  `gather` (optional) picks the input row of each
 // output row, so the last norm runs on the wanted rows only.  With `residual`

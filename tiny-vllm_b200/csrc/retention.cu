@@ -35,6 +35,15 @@
 #define RET_PAIR_INTERLEAVED 0
 #define RET_PAIR_HALF_SPLIT 1
 #define RET_MAX_TURNED 512        // pairs of a head that turn: sine and cosine of a token in shared memory
+#define RET_ACT_NONE 0
+#define RET_ACT_SILU 1
+#define RET_ACT_SIGMOID 2
+
+// what an output is multiplied by: silu(z), sigmoid(z) or z itself
+__device__ __forceinline__ float output_gate(float z, int act) {
+    const float sig = __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z)));
+    return act == RET_ACT_SILU ? __fmul_rn(z, sig) : act == RET_ACT_SIGMOID ? sig : z;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(128) retention_prepare_kernel(
@@ -418,43 +427,67 @@ __global__ void __launch_bounds__(128) retention_gate_prefix_kernel(
     }
 }
 
-// What a recurrence with a gate a channel reads, from a packed projection: q = act(projection) (act none or SiLU)
-// and g = lower + (1 - lower) * sigmoid(projection + bias), a gate that never falls below `lower`; both float32
-// [tokens, per].  `bias` and `lower` (float32 [per]) may be null: 0.
+// What a recurrence with a gate a channel reads, from a packed projection: q = act(projection) * q_scale (act none
+// or SiLU) and g = lower + (1 - lower) * sigmoid(projection + bias)^gate_exponent, a gate that never falls below
+// `lower`; and, with k_out, the keys as projected; all float32 [tokens, per].  `bias` and `lower` (float32 [per])
+// may be null: 0.  With `gate_pre` (float32 [tokens, per]) the gates' pre-activations come from there.
+__device__ __forceinline__ float gate_value(float z, float exponent) {
+    if (exponent == 1.0f) return __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z)));
+    // sigmoid(z)^e = exp(-e ln(1 + exp(-z))), the logarithm taken so that it loses nothing at either end
+    return expf(-__fmul_rn(exponent, __fadd_rn(fmaxf(-z, 0.0f), log1pf(expf(-fabsf(z))))));
+}
+
+struct GateArgs {
+    const float* bias;
+    const float* lower;
+    const float* gate_pre;
+    int q_act;
+    float q_scale, gate_exponent;
+};
+
+__device__ __forceinline__ float query_value(float x, const GateArgs& a) {
+    return __fmul_rn(a.q_act ? __fdiv_rn(x, __fadd_rn(1.0f, expf(-x))) : x, a.q_scale);
+}
+__device__ __forceinline__ float bounded_gate(float z, const GateArgs& a, int e) {
+    if (a.bias) z = __fadd_rn(z, a.bias[e]);
+    const float low = a.lower ? a.lower[e] : 0.0f;
+    return __fmaf_rn(__fsub_rn(1.0f, low), gate_value(z, a.gate_exponent), low);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) gated_prepare_kernel(
-    const T* __restrict__ proj, int64_t token_stride, int q_at, int g_at, int per, const float* __restrict__ bias,
-    const float* __restrict__ lower, int q_act, float* __restrict__ q_out, float* __restrict__ g_out) {
+    const T* __restrict__ proj, int64_t token_stride, int q_at, int g_at, int k_at, int per, GateArgs args,
+    float* __restrict__ q_out, float* __restrict__ g_out, float* __restrict__ k_out) {
     const int token = blockIdx.y;
     const int e = blockIdx.x * blockDim.x + threadIdx.x;
     if (e >= per) return;
     const T* row = proj + (int64_t)token * token_stride;
-    const float x = to_float<T>(row[q_at + e]);
-    q_out[(int64_t)token * per + e] = q_act ? __fdiv_rn(x, __fadd_rn(1.0f, expf(-x))) : x;
-    float z = to_float<T>(row[g_at + e]);
-    if (bias) z = __fadd_rn(z, bias[e]);
-    const float sig = __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z)));
-    const float low = lower ? lower[e] : 0.0f;
-    g_out[(int64_t)token * per + e] = __fmaf_rn(__fsub_rn(1.0f, low), sig, low);
+    const int64_t at = (int64_t)token * per + e;
+    q_out[at] = query_value(to_float<T>(row[q_at + e]), args);
+    g_out[at] = bounded_gate(args.gate_pre ? args.gate_pre[at] : to_float<T>(row[g_at + e]), args, e);
+    if (k_out) k_out[at] = to_float<T>(row[k_at + e]);
 }
 
-extern "C" int tvb_gated_prepare(const void* proj, long long token_stride, int q_at, int g_at, int per,
-                                 const float* bias, const float* lower, int q_act, float* q_out, float* g_out,
-                                 int tokens, int dtype, void* stream) {
+extern "C" int tvb_gated_prepare(const void* proj, long long token_stride, int q_at, int g_at, int k_at, int per,
+                                 const float* bias, const float* lower, const float* gate_pre, int q_act, float q_scale,
+                                 float gate_exponent, float* q_out, float* g_out, float* k_out, int tokens, int dtype,
+                                 void* stream) {
     if (tokens <= 0) return 0;
-    if (per <= 0 || q_at < 0 || g_at < 0 || !q_out || !g_out) return TVB_BAD_ARGUMENT;
+    if (per <= 0 || q_at < 0 || (g_at < 0 && !gate_pre) || (k_out && k_at < 0) || !q_out || !g_out) return TVB_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     for (int first = 0; first < tokens; first += 65535) {
         const int count = min(65535, tokens - first);
         const dim3 grid((per + 255) / 256, count);
+        const int64_t done = (int64_t)first * per;
+        const GateArgs args{bias, lower, gate_pre ? gate_pre + done : nullptr, q_act, q_scale, gate_exponent};
         if (dtype == TVB_F32)
             gated_prepare_kernel<float><<<grid, 256, 0, s>>>((const float*)proj + (int64_t)first * token_stride, token_stride,
-                                                            q_at, g_at, per, bias, lower, q_act, q_out + (int64_t)first * per,
-                                                            g_out + (int64_t)first * per);
+                                                            q_at, g_at, k_at, per, args, q_out + done, g_out + done,
+                                                            k_out ? k_out + done : nullptr);
         else if (dtype == TVB_BF16)
             gated_prepare_kernel<bf16><<<grid, 256, 0, s>>>((const bf16*)proj + (int64_t)first * token_stride, token_stride,
-                                                           q_at, g_at, per, bias, lower, q_act, q_out + (int64_t)first * per,
-                                                           g_out + (int64_t)first * per);
+                                                           q_at, g_at, k_at, per, args, q_out + done, g_out + done,
+                                                           k_out ? k_out + done : nullptr);
         else return TVB_BAD_ARGUMENT;
     }
     return tvb_last_error();
@@ -463,21 +496,25 @@ extern "C" int tvb_gated_prepare(const void* proj, long long token_stride, int q
 // One token a request (a decode step) of the recurrence with a gate a channel, the whole mixer between its two
 // projections in one launch: a CTA a (request, head) reads the token's q, gate and v from the packed projection
 // (q = act(q), g = lower + (1 - lower) sigmoid(g + bias), as gated_prepare), moves the head's state once,
-// S <- diag(g) S + (1 - g) v^T, sums o = S^T q on the way, divides o by its root mean square (with `unit_norm`),
-// multiplies by `norm_weight` and rounds once.  A thread owns VEC neighbouring columns of the state and one of
+// S <- diag(g) S + (1 - g) v^T (with k_at >= 0: + k v^T), sums o = S^T q on the way, divides o by its root mean
+// square (with `unit_norm`), multiplies by `norm_weight`, gates by act(projection from `out_gate_at` on) and rounds
+// once.  With `low_at` >= 0 the gates' pre-activations are a product done here: `rank` numbers of the row from
+// `low_at` on times the rows of `low_weight` [heads * dim, rank] (rank a multiple of 8).  A thread owns VEC neighbouring columns of the state and one of
 // SLICES slices of its rows; the slices' partial sums meet in shared memory in the order of the slices.
 #define STEP_THREADS 256
 template <typename T, int VEC>
 __global__ void __launch_bounds__(STEP_THREADS) gated_step_kernel(
-    const T* proj, int64_t token_stride, int q_at, int g_at, int v_at, const float* __restrict__ bias,
-    const float* __restrict__ lower, int q_act, float* __restrict__ state, const int* __restrict__ row_starts,
+    const T* proj, int64_t token_stride, int q_at, int g_at, int k_at, int v_at, int low_at, int rank,
+    const T* __restrict__ low_weight, GateArgs args, float* __restrict__ state, const int* __restrict__ row_starts,
     const int* __restrict__ state_slots, const int* __restrict__ token_row, const float* __restrict__ norm_weight,
-    int unit_norm, float eps, T* __restrict__ out, int64_t out_stride, int heads, int dim, int vdim) {
+    int unit_norm, float eps, int out_gate_at, int out_act, T* __restrict__ out, int64_t out_stride, int heads, int dim,
+    int vdim) {
     extern __shared__ __align__(16) float step_shared[];
     __shared__ float scratch[32];
     float* q_s = step_shared;                     // [dim]
     float* g_s = q_s + dim;                       // [dim]
-    float* o_s = g_s + dim;                       // [slices][columns rounded up to VEC]
+    float* k_s = g_s + dim;                       // [dim]
+    float* o_s = k_s + dim;                       // [slices][columns rounded up to VEC]
     const int row = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
     const int token = row_starts[row];
     T* dst = out + (int64_t)token * out_stride + (int64_t)head * vdim;
@@ -488,13 +525,14 @@ __global__ void __launch_bounds__(STEP_THREADS) gated_step_kernel(
     const T* src = proj + (int64_t)token * token_stride;
     for (int d = tid; d < dim; d += STEP_THREADS) {
         const int e = head * dim + d;
-        const float x = to_float<T>(src[q_at + e]);
-        q_s[d] = q_act ? __fdiv_rn(x, __fadd_rn(1.0f, expf(-x))) : x;
-        float z = to_float<T>(src[g_at + e]);
-        if (bias) z = __fadd_rn(z, bias[e]);
-        const float sig = __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z)));
-        const float low = lower ? lower[e] : 0.0f;
-        g_s[d] = __fmaf_rn(__fsub_rn(1.0f, low), sig, low);
+        q_s[d] = query_value(to_float<T>(src[q_at + e]), args);
+        float z = 0.0f;
+        if (low_at >= 0) {
+            for (int r = 0; r < rank; ++r)
+                z = __fmaf_rn(to_float<T>(src[low_at + r]), to_float<T>(low_weight[(int64_t)e * rank + r]), z);
+        } else z = args.gate_pre ? args.gate_pre[(int64_t)token * heads * dim + e] : to_float<T>(src[g_at + e]);
+        g_s[d] = bounded_gate(z, args, e);
+        k_s[d] = k_at >= 0 ? to_float<T>(src[k_at + e]) : __fsub_rn(1.0f, g_s[d]);
     }
     __syncthreads();
     const int groups = (vdim + VEC - 1) / VEC;    // groups of VEC columns
@@ -526,7 +564,7 @@ __global__ void __launch_bounds__(STEP_THREADS) gated_step_kernel(
 #pragma unroll
             for (int u = 0; u < 4; ++u)
                 if (d0 + u < last) {
-                    const float g = g_s[d0 + u], k = __fsub_rn(1.0f, g), q = q_s[d0 + u];
+                    const float g = g_s[d0 + u], k = k_s[d0 + u], q = q_s[d0 + u];
 #pragma unroll
                     for (int j = 0; j < VEC; ++j) {
                         s[u][j] = __fmaf_rn(k, vv[j], __fmul_rn(g, s[u][j]));
@@ -556,18 +594,21 @@ __global__ void __launch_bounds__(STEP_THREADS) gated_step_kernel(
     for (int c = tid; c < vdim; c += STEP_THREADS) {
         float x = __fmul_rn(o_s[c], factor);
         if (norm_weight) x = __fmul_rn(x, norm_weight[c]);
+        if (out_gate_at >= 0) x = __fmul_rn(x, output_gate(to_float<T>(src[out_gate_at + head * vdim + c]), out_act));
         dst[c] = from_float<T>(x);
     }
 }
 
 // proj [rows of one token each, columns] of the storage type; state float32 [slots, heads, dim, vdim]; every entry
 // of row_starts [rows + 1] holds one token; out [tokens, heads * vdim] of the storage type.
-extern "C" int tvb_gated_step(const void* proj, long long token_stride, int q_at, int g_at, int v_at, const float* bias,
-                              const float* lower, int q_act, float* state, const int* row_starts,
-                              const int* state_slots, const int* token_row, const float* norm_weight, int unit_norm,
-                              float eps, void* out, long long out_stride, int rows, int heads, int dim, int vdim,
-                              int dtype, void* stream) {
+extern "C" int tvb_gated_step(const void* proj, long long token_stride, int q_at, int g_at, int k_at, int v_at, int low_at,
+                              int rank, const void* low_weight, const float* bias, const float* lower,
+                              const float* gate_pre, int q_act, float q_scale, float gate_exponent, float* state,
+                              const int* row_starts, const int* state_slots, const int* token_row,
+                              const float* norm_weight, int unit_norm, float eps, int out_gate_at, int out_act, void* out,
+                              long long out_stride, int rows, int heads, int dim, int vdim, int dtype, void* stream) {
     if (rows <= 0) return 0;
+    if ((low_at >= 0 && (!low_weight || rank <= 0)) || (low_at < 0 && !gate_pre && g_at < 0)) return TVB_BAD_ARGUMENT;
     if (heads <= 0 || heads > 65535 || dim <= 0 || dim > 256 || vdim <= 0 || vdim > 4 * STEP_THREADS || !state)
         return TVB_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
@@ -575,21 +616,19 @@ extern "C" int tvb_gated_step(const void* proj, long long token_stride, int q_at
     const int vec = by_four ? 4 : 1;
     if (!by_four && vdim > STEP_THREADS) return TVB_BAD_ARGUMENT;
     const int groups = (vdim + vec - 1) / vec, slices = STEP_THREADS / groups > 0 ? STEP_THREADS / groups : 1;
-    const size_t smem = (size_t)(2 * dim + slices * groups * vec) * sizeof(float);
+    const size_t smem = (size_t)(3 * dim + slices * groups * vec) * sizeof(float);
+    const GateArgs args{bias, lower, gate_pre, q_act, q_scale, gate_exponent};
     const dim3 grid(rows, heads);
 #define GO(T, V) gated_step_kernel<T, V><<<grid, STEP_THREADS, smem, s>>>(                                          \
-        (const T*)proj, token_stride, q_at, g_at, v_at, bias, lower, q_act, state, row_starts, state_slots, token_row, \
-        norm_weight, unit_norm, eps, (T*)out, out_stride, heads, dim, vdim)
+        (const T*)proj, token_stride, q_at, g_at, k_at, v_at, low_at, rank, (const T*)low_weight, args, state,        \
+        row_starts, state_slots, token_row, norm_weight, unit_norm, eps, out_gate_at, out_act, (T*)out, out_stride,  \
+        heads, dim, vdim)
     if (dtype == TVB_F32) { if (by_four) GO(float, 4); else GO(float, 1); }
     else if (dtype == TVB_BF16) { if (by_four) GO(bf16, 4); else GO(bf16, 1); }
     else return TVB_BAD_ARGUMENT;
 #undef GO
     return tvb_last_error();
 }
-
-#define RET_ACT_NONE 0
-#define RET_ACT_SILU 1
-#define RET_ACT_SIGMOID 2
 
 // A warp a (token, head): o / sqrt(mean(o^2) + eps) (with `unit_norm`; times `norm_weight` [vdim], one for all
 // heads, if given), times act(gate).
@@ -614,11 +653,7 @@ __global__ void __launch_bounds__(128) retention_finish_kernel(
     for (int i = lane; i < vdim; i += 32) {
         float x = __fmul_rn(src[i], factor);
         if (norm_weight) x = __fmul_rn(x, norm_weight[i]);
-        if (g) {
-            const float z = to_float<T>(g[i]);
-            const float sig = __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z)));
-            x = __fmul_rn(x, act == RET_ACT_SILU ? __fmul_rn(z, sig) : act == RET_ACT_SIGMOID ? sig : z);
-        }
+        if (g) x = __fmul_rn(x, output_gate(to_float<T>(g[i]), act));
         dst[i] = from_float<T>(x);
     }
 }

@@ -14,7 +14,7 @@ import torch
 
 from ..config.spec import ModelSpec
 from ..parts import BuildContext, build_part
-from ..parts.base import Part
+from ..parts.base import EMBEDDING, Part
 from ..weights.loader import bind_tensors, load_checkpoint
 from ..weights.random_init import random_tensors
 
@@ -52,6 +52,12 @@ class Model:
     def cache_needs(self) -> list:
         """What each entry of the run list needs of the cache."""
         return [self.blocks[step.layer].cache_need() for step in self.order]
+
+    def other_states(self) -> dict:
+        """Per-request states that belong to no run: what the embedding carries from token to token."""
+        asked = getattr(self.embedding, "state_need", None)
+        need = asked() if asked is not None else None
+        return {} if need is None else {EMBEDDING: need}
 
     def cache_sources(self) -> list:
         return [step.cache_from for step in self.order]
@@ -112,7 +118,8 @@ class Model:
     def forward(self, ctx) -> torch.Tensor | None:
         """Logits (float32, [wanted rows, vocab]) of the step described by ``ctx``,
         or None when no row is wanted.  Keys and values of all tokens are written."""
-        hidden = self.embedding.forward(ctx.token_ids)
+        embed = getattr(self.embedding, "forward_step", None)
+        hidden = embed(ctx) if embed is not None else self.embedding.forward(ctx.token_ids)
         residual = None
         for run, step in enumerate(self.order):
             hidden, residual = self.blocks[step.layer].forward(hidden, residual, ctx, run)

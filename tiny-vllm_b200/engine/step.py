@@ -138,7 +138,8 @@ class StepRunner:
         self.manager = CacheManager(groups, page_size, list(num_pages), max_requests)
         self.storage = CacheStorage(groups, where, needs, page_size=page_size,
                                     pages_per_group=list(num_pages), num_state_slots=max_requests,
-                                    dtype=self.dtype, device=self.device)
+                                    dtype=self.dtype, device=self.device,
+                                    other_states=getattr(model, "other_states", dict)())
         self.vocab_size = model.spec.vocab_size
         self._pinned: torch.Tensor | None = None
         self._pinned_free: torch.cuda.Event | None = None

@@ -276,6 +276,7 @@ def windowed_attention(ctx, mixer, projected: torch.Tensor, at: int, run: int, o
     g_at = k_at + mixer.k_cols + mixer.v_cols
     v_here = projected[:, v_at:v_at + mixer.num_kv_heads * mixer.value_dim]
     q_bias, k_bias = getattr(mixer, "q_bias", None), getattr(mixer, "k_bias", None)
+    v_bias = getattr(mixer, "v_bias", None)
     bias_table, segment = getattr(mixer, "bias_table", None), getattr(mixer, "segment", None)
     if values_are_keys and not writes:
         raise kernels.KernelError("values that are the keys need the step's keys written to the cache")
@@ -321,13 +322,13 @@ def windowed_attention(ctx, mixer, projected: torch.Tensor, at: int, run: int, o
             pairing="interleaved" if position is None else position.pairing,
             slots=ctx.slots[group] if writes else None, key_cache=keys, value_cache=values,
             v_first=v_first, blend=mixer.vmix if v_first is not None else None,
-            q_bias=q_bias, k_bias=k_bias, v_bias=k_bias if values_are_keys else None)
+            q_bias=q_bias, k_bias=k_bias, v_bias=k_bias if values_are_keys else v_bias)
     gate = projected[:, g_at:g_at + mixer.gate_cols] if mixer.gate else None
     queries = projected[:, q_at:q_at + mixer.q_cols]
     heads = dict(num_q=mixer.num_heads, num_kv=mixer.num_kv_heads, key_dim=mixer.key_dim,
                  value_dim=mixer.value_dim, window=mixer.window, keep_first=mixer.keep_first, scale=mixer.scale,
                  gate_per_head=mixer.gate == "head", slopes=mixer.slopes, sinks=mixer.sinks,
-                 bias_table=bias_table, segment=segment)
+                 bias_table=bias_table, segment=segment, softcap=getattr(mixer, "softcap", None))
     if not (segment and mixer.window) and windowed_on_tensor_cores(mixer, projected, q_at, g_at, out):
         # bfloat16: prompt portions in tiles of 64 tokens, single tokens (decoded ones, whose keys are in the
         # cache by now) one CTA per kv head and chunk of keys
@@ -359,7 +360,7 @@ def windowed_attention(ctx, mixer, projected: torch.Tensor, at: int, run: int, o
         ctx.token_row, ctx.positions, num_q=mixer.num_heads, num_kv=mixer.num_kv_heads, head_dim=mixer.key_dim,
         value_dim=mixer.value_dim, window=mixer.window, keep_first=mixer.keep_first, scale=mixer.scale,
         gate=gate, gate_per_head=mixer.gate == "head", slopes=mixer.slopes, sinks=mixer.sinks, out=out,
-        scratch=scratch, max_chunks=ctx.split_chunks, bias_table=bias_table, segment=segment)
+        scratch=scratch, max_chunks=ctx.split_chunks, bias_table=bias_table, segment=segment, softcap=getattr(mixer, "softcap", None))
 
 
 def latent_attention(ctx, mixer, projected: torch.Tensor, run: int) -> torch.Tensor:

@@ -135,6 +135,39 @@ def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor | None 
 
 
 # -------------------------------------------------------------------- RMSNorm
+def embed_pairs(table: torch.Tensor, ids: torch.Tensor, *, positions: torch.Tensor, token_row: torch.Tensor,
+                row_starts: torch.Tensor, state_slots: torch.Tensor, pairs: dict | None = None) -> torch.Tensor:
+    """float32 [tokens, width]: table[ids[t]], plus, with ``pairs`` (``table`` [buckets + 1, width], ``mul_prev``,
+    ``mul_cur``, ``state`` int32 [slots, 1]), the pair row (previous * mul_prev + ids[t] * mul_cur) mod buckets, or
+    the last row at position 0.  The token before an entry's first one is read from the state of the entry's
+    slot, which is left as the entry's last token."""
+    _need_cuda(table, ids, positions, token_row, row_starts, state_slots)
+    tokens, rows = ids.shape[0], state_slots.shape[0]
+    if table.dim() != 2 or not table.is_contiguous():
+        raise KernelError("embed_pairs wants a contiguous [vocab, width] table")
+    for name, t, shape in (("ids", ids, (tokens,)), ("positions", positions, (tokens,)),
+                           ("token_row", token_row, (tokens,)), ("row_starts", row_starts, (rows + 1,)),
+                           ("state_slots", state_slots, (rows,))):
+        if t.dtype != torch.int32 or t.shape != shape or not t.is_contiguous():
+            raise KernelError(f"embed_pairs: {name} must be contiguous int32 {list(shape)}")
+    (vocab, width), hashed, state, buckets, mul_prev, mul_cur = table.shape, None, None, 0, 0, 0
+    if pairs is not None:
+        hashed, state, mul_prev, mul_cur = pairs["table"], pairs["state"], pairs["mul_prev"], pairs["mul_cur"]
+        _need_cuda(hashed, state)
+        if hashed.dim() != 2 or hashed.shape[1] != width or hashed.shape[0] < 2 or hashed.dtype != table.dtype \
+                or not hashed.is_contiguous():
+            raise KernelError("embed_pairs: the pair table is contiguous [buckets + 1, width] of the table's dtype")
+        if state.dtype != torch.int32 or state.dim() != 2 or state.shape[1] != 1 or not state.is_contiguous():
+            raise KernelError("embed_pairs: the state is contiguous int32 [slots, 1]")
+        buckets = hashed.shape[0] - 1
+    out = torch.empty((tokens, width), dtype=torch.float32, device=table.device)
+    fn = _fn("pointwise", "tvb_embed_pairs", [c_void_p] * 9 + [c_int] * 7 + [c_void_p])
+    _check(fn(table.data_ptr(), _ptr(hashed), ids.data_ptr(), positions.data_ptr(), token_row.data_ptr(),
+              row_starts.data_ptr(), state_slots.data_ptr(), _ptr(state), out.data_ptr(), tokens, width, vocab, buckets,
+              mul_prev, mul_cur, dtype_tag(table.dtype), _stream()), "embed_pairs")
+    return out
+
+
 def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, *, residual: torch.Tensor | None = None,
              rows: torch.Tensor | None = None, out: torch.Tensor | None = None,
              residual_out: torch.Tensor | None = None, want_residual: bool = True):
@@ -303,7 +336,7 @@ def attention_rows(q: torch.Tensor, q_token_stride: int, key_cache: torch.Tensor
                    gate: torch.Tensor | None = None, gate_per_head: bool = False,
                    slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
                    value_offset: int | None = None, bias_table: torch.Tensor | None = None,
-                   segment: int | None = None) -> torch.Tensor:
+                   segment: int | None = None, softcap: float | None = None) -> torch.Tensor:
     """Paged causal attention, one warp per (token, head).
 
     ``q`` holds the query heads of token t at ``t * q_token_stride`` elements
@@ -318,7 +351,8 @@ def attention_rows(q: torch.Tensor, q_token_stride: int, key_cache: torch.Tensor
     softmax's denominator once.  ``value_offset``: the values are the ``value_dim`` elements from
     there on of every key row (``value_cache`` is then None).  ``bias_table`` (float32 [rows, num_q]):
     table[min(position - j, rows - 1), head] is added to the score of key j; ``segment``: the query at
-    position p sees only the keys from p - p % segment on."""
+    position p sees only the keys from p - p % segment on.  ``softcap``: the scaled score s becomes softcap *
+    tanh(s / softcap), before any bias."""
     _need_cuda(q, key_cache, value_cache, block_tables, token_row, positions, scratch, gate, slopes, sinks,
                bias_table)
     if bias_table is not None and (bias_table.dtype != torch.float32 or bias_table.dim() != 2
@@ -367,7 +401,7 @@ def attention_rows(q: torch.Tensor, q_token_stride: int, key_cache: torch.Tensor
     fn = _fn("attention_rows", "tvb_attention_rows_masked",
              [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
               c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int,
-              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
+              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p])
     _check(fn(q.data_ptr(), q_token_stride, key_cache.data_ptr(), value_ptr, value_stride,
               block_tables.data_ptr(), block_tables.shape[1], token_row.data_ptr(),
               positions.data_ptr(), out.data_ptr(), out.stride(0), _ptr(gate),
@@ -375,7 +409,7 @@ def attention_rows(q: torch.Tensor, q_token_stride: int, key_cache: torch.Tensor
               _ptr(bias_table), 0 if bias_table is None else bias_table.shape[0], segment or 0,
               _ptr(scratch), max_chunks, tokens, num_q, num_kv,
               head_dim, value_dim, key_cache.shape[2], window or 0, keep_first if window else 0, scale,
-              dtype_tag(q.dtype), _stream()),
+              softcap or 0.0, dtype_tag(q.dtype), _stream()),
            "attention_rows", 2 if max_chunks > 0 else 1)
     return out
 
@@ -870,6 +904,235 @@ def route_softmax_gated(logits: torch.Tensor, proj: torch.Tensor, *, experts: in
     return out, passed
 
 
+# ------------------------------------------------ a residual of several float32 streams
+HYPER_MAX_STREAMS = 32
+
+
+def _pair_checks(who: str, y, tokens: int, width: int) -> None:
+    if y.left.shape != (tokens, width) or y.right.shape != (tokens, width) or y.left.dtype != y.right.dtype \
+            or not y.left.is_contiguous() or not y.right.is_contiguous():
+        raise KernelError(f"{who}: a pair is two contiguous [tokens, width] tensors of one dtype")
+    for t in (y.left_weight, y.right_weight, y.left_bias, y.right_bias):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (width,) or not t.is_contiguous()):
+            raise KernelError(f"{who}: a pair's weights and biases are contiguous float32 [width]")
+    if y.left_weight is None or y.right_weight is None:
+        raise KernelError(f"{who}: a pair's norms have weights")
+    _need_cuda(y.left, y.right, y.left_weight, y.right_weight, y.left_bias, y.right_bias)
+
+
+def hyper_norm(stream: torch.Tensor, *, streams: int, w_in: torch.Tensor | None, weight: torch.Tensor,
+               bias: torch.Tensor, eps: float, out_dtype: torch.dtype, y=None, w_mix: torch.Tensor | None = None,
+               w_out: torch.Tensor | None = None, rows: torch.Tensor | None = None):
+    """The write behind a sublayer and the norm in front of the next, over a residual of several float32 streams.
+
+    ``stream`` [tokens, streams, width], or [tokens, width] while all streams are equal.  With ``y`` x'_t = sum_s
+    w_mix[s, t] x_s + w_out[t] y for all streams at once (written back; a new tensor where the streams were one), y
+    being [tokens, width] or a pair (``left``, ``right`` with norm weights, optional biases, ``eps`` and ``factor``:
+    factor * (left / rms(left) * left_weight + right / rms(right) * right_weight)).  Then u = sum_t w_in[t] x'_t
+    (w_in None: the plain sum) and v = (u - mean) / sqrt(mean squared deviation + eps) * weight + bias, rounded once
+    to ``out_dtype``.  All float32.  Returns (v, streams).  With ``rows`` (int32) only those rows of v are
+    produced and nothing is written: (v, None)."""
+    _need_cuda(stream, w_in, weight, bias, w_mix, w_out, rows)
+    spread = stream.dim() == 2
+    if stream.dtype != torch.float32 or not stream.is_contiguous() or stream.dim() not in (2, 3) or (
+            not spread and stream.shape[1] != streams):
+        raise KernelError("hyper_norm wants contiguous float32 streams [tokens, streams, width] or [tokens, width]")
+    tokens, width = stream.shape[0], stream.shape[-1]
+    if not 0 < streams <= HYPER_MAX_STREAMS:
+        raise KernelError(f"hyper_norm takes up to {HYPER_MAX_STREAMS} streams, not {streams}")
+    for name, t, shape in (("w_in", w_in, (streams,)), ("w_out", w_out, (streams,)), ("w_mix", w_mix, (streams, streams)),
+                           ("weight", weight, (width,)), ("bias", bias, (width,))):
+        if t is not None and (t.dtype != torch.float32 or t.shape != shape or not t.is_contiguous()):
+            raise KernelError(f"hyper_norm: {name} must be contiguous float32 {list(shape)}")
+    if rows is not None and rows.dtype != torch.int32:
+        raise KernelError("hyper_norm: rows must be int32")
+    left = right = None
+    weights, pair_eps, factor = [None] * 4, 0.0, 1.0
+    if y is not None:
+        if w_mix is None or w_out is None:
+            raise KernelError("hyper_norm: a write needs the mixing matrix and the shares of the streams")
+        if isinstance(y, torch.Tensor):
+            if y.shape != (tokens, width) or not y.is_contiguous():
+                raise KernelError("hyper_norm: y must be contiguous [tokens, width]")
+            _need_cuda(y)
+            left = y
+        else:
+            _pair_checks("hyper_norm", y, tokens, width)
+            left, right, pair_eps, factor = y.left, y.right, y.eps, y.factor
+            weights = [y.left_weight, y.right_weight, y.left_bias, y.right_bias]
+    if width * 4 * (3 if right is not None else 1) > 200 * 1024:
+        raise KernelError(f"hyper_norm: width {width} is larger than a row buffer of shared memory holds")
+    count = tokens if rows is None else rows.shape[0]
+    out = torch.empty((count, width), dtype=out_dtype, device=stream.device)
+    updated = None
+    if rows is None:
+        updated = stream
+        if left is not None and spread:
+            updated = torch.empty((tokens, streams, width), dtype=torch.float32, device=stream.device)
+    fn = _fn("hyper_streams", "tvb_hyper_norm",
+             [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float,
+              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+              c_float, c_int, c_void_p])
+    _check(fn(stream.data_ptr(), 1 if spread else 0, _ptr(left), _ptr(right),
+              dtype_tag(left.dtype) if left is not None else F32, *(_ptr(t) for t in weights), pair_eps, factor,
+              _ptr(w_mix), _ptr(w_out), _ptr(w_in), weight.data_ptr(), bias.data_ptr(), out.data_ptr(),
+              dtype_tag(out_dtype), _ptr(updated) if left is not None else None, _ptr(rows), count, streams, width, eps,
+              _pdl("norm"), _stream()), "hyper_norm")
+    if updated is not None and y is not None:
+        updated.pending = None
+    return out, updated
+
+
+def normed_pair_sum(y) -> torch.Tensor:
+    """float32 [tokens, width]: factor * (left / rms(left) * left_weight + right / rms(right) * right_weight) of a pair
+    (as :func:`hyper_norm` takes it)."""
+    tokens, width = y.left.shape
+    _pair_checks("normed_pair_sum", y, tokens, width)
+    if width * 8 > 200 * 1024:
+        raise KernelError(f"normed_pair_sum: width {width} is larger than a row buffer of shared memory holds")
+    out = torch.empty((tokens, width), dtype=torch.float32, device=y.left.device)
+    fn = _fn("hyper_streams", "tvb_normed_pair_sum",
+             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int,
+              c_int, c_void_p])
+    _check(fn(y.left.data_ptr(), y.right.data_ptr(), dtype_tag(y.left.dtype), y.left_weight.data_ptr(),
+              y.right_weight.data_ptr(), _ptr(y.left_bias), _ptr(y.right_bias), y.eps, y.factor, out.data_ptr(), tokens,
+              width, _stream()), "normed_pair_sum")
+    return out
+
+
+def add_row_bias(y: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """y[t] += bias in place (float32 bias [width], the sum in float32); returns y."""
+    _need_cuda(y, bias)
+    if y.dim() != 2 or not y.is_contiguous() or bias.dtype != torch.float32 or bias.shape != (y.shape[1],) \
+            or not bias.is_contiguous():
+        raise KernelError("add_row_bias wants contiguous [tokens, width] and a float32 bias [width]")
+    fn = _fn("hyper_streams", "tvb_add_row_bias", [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(fn(y.data_ptr(), bias.data_ptr(), y.shape[0], y.shape[1], dtype_tag(y.dtype), _stream()), "add_row_bias")
+    return y
+
+
+# ------------------------------------------------ short convolution and selective scan
+CONV_TAPS = (2, 4, 8, 16, 32)     # what the kernel is compiled for: fewer taps are padded with zeros in front
+CONV_ACTS = {None: 0, "silu": 1}
+SCAN_MAX_STATE = 256
+STEP_FUSED_ROWS = 16              # rows up to which the step kernel does the step sizes' product itself
+STEP_FUSED_MAX_RANK = 1024
+
+
+def _entry_checks(who: str, tokens: int, row_starts, state_slots, token_row) -> int:
+    rows = state_slots.shape[0]
+    for name, t, shape in (("row_starts", row_starts, (rows + 1,)), ("state_slots", state_slots, (rows,)),
+                           ("token_row", token_row, (tokens,))):
+        if t.dtype != torch.int32 or t.shape != shape or not t.is_contiguous():
+            raise KernelError(f"{who}: {name} must be contiguous int32 {list(shape)}")
+    return rows
+
+
+def short_convolution(x: torch.Tensor, taps: torch.Tensor, *, bias: torch.Tensor | None, act: str | None,
+                      state: torch.Tensor, row_starts: torch.Tensor, state_slots: torch.Tensor,
+                      token_row: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """act(bias + sum_j taps[j] * x[t - (K - 1) + j]) per channel: x [tokens, channels] (rows may be strided), taps
+    float32 [K, channels] with K one of CONV_TAPS (the last tap is the current token's).  The inputs before an
+    entry's first token are those ``state`` (float32 [slots, K - 1, channels], oldest first) keeps in the entry's
+    slot, which is left as the entry's last K - 1 inputs."""
+    _need_cuda(x, taps, bias, state, row_starts, state_slots, token_row, out)
+    tokens, channels = x.shape
+    rows = _entry_checks("short_convolution", tokens, row_starts, state_slots, token_row)
+    if x.stride(1) != 1 or taps.dim() != 2 or taps.shape[0] not in CONV_TAPS or taps.shape[1] != channels \
+            or taps.dtype != torch.float32 or not taps.is_contiguous():
+        raise KernelError(f"short_convolution wants x with contiguous rows and float32 taps [{CONV_TAPS}, channels]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (channels,) or not bias.is_contiguous()):
+        raise KernelError("short_convolution: the bias is contiguous float32 [channels]")
+    if state.dtype != torch.float32 or state.dim() != 3 or state.shape[1:] != (taps.shape[0] - 1, channels) \
+            or not state.is_contiguous():
+        raise KernelError("short_convolution: the state is contiguous float32 [slots, K - 1, channels]")
+    if act not in CONV_ACTS:
+        raise KernelError(f"short_convolution: the activation is None or 'silu', not {act!r}")
+    if out is None:
+        out = torch.empty((tokens, channels), dtype=x.dtype, device=x.device)
+    elif out.shape != x.shape or out.dtype != x.dtype or out.stride(1) != 1:
+        raise KernelError("short_convolution: out must be [tokens, channels] of the dtype of x")
+    fn = _fn("short_conv", "tvb_short_conv",
+             [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+              c_longlong, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(x.data_ptr(), x.stride(0), taps.data_ptr(), taps.shape[0], _ptr(bias), CONV_ACTS[act], state.data_ptr(),
+              row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows,
+              tokens, channels, dtype_tag(x.dtype), _stream()), "short_convolution")
+    return out
+
+
+def selective_step_takes(rows: int, rank: int) -> bool:
+    """Whether a step of single tokens does the step sizes' low-rank product inside the step kernel (every CTA reads
+    the weights of its channels for its own request: for few requests that is cheaper than a launch)."""
+    return rows <= STEP_FUSED_ROWS and rank % 8 == 0 and 0 < rank <= STEP_FUSED_MAX_RANK
+
+
+def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor, b: torch.Tensor, c: torch.Tensor,
+                   a: torch.Tensor, d: torch.Tensor, dt_bias: torch.Tensor | None, state: torch.Tensor,
+                   row_starts: torch.Tensor, state_slots: torch.Tensor, token_row: torch.Tensor, out: torch.Tensor,
+                   single: bool = False, low: torch.Tensor | None = None, dt_weight: torch.Tensor | None = None,
+                   lanes: int = 0) -> torch.Tensor:
+    """The selective scan between its projections: dt = softplus(pre + dt_bias), S <- exp(dt A) S + dt x B^T, y = S C +
+    D x, out = y silu(z), token by token from the float32 ``state`` [slots, channels, n] of the entry's slot, which
+    is left as the state after the entry's last token.
+
+    ``x``, ``z``, ``out`` [tokens, channels] and ``b``, ``c`` [tokens, n] of the storage type (rows may be strided;
+    b and c alike), ``pre`` float32 [tokens, channels], ``a`` float32 [channels, n], ``d`` and ``dt_bias`` float32
+    [channels].  ``single``: every entry is one token, one launch that reads and writes the state once; instead of
+    ``pre`` it may take ``low`` [tokens, rank] (rows apart as those of b) and ``dt_weight`` [channels, rank] and do the
+    product itself.  ``lanes`` (2, 4, 8, 16; 0: chosen): the lanes of a scan that share a channel."""
+    _need_cuda(x, pre, z, b, c, a, d, dt_bias, state, row_starts, state_slots, token_row, out, low, dt_weight)
+    tokens, channels = x.shape
+    n = a.shape[1]
+    rows = _entry_checks("selective_scan", tokens, row_starts, state_slots, token_row)
+    for name, t, shape in (("z", z, (tokens, channels)), ("out", out, (tokens, channels)), ("b", b, (tokens, n)),
+                           ("c", c, (tokens, n))):
+        if t.shape != shape or t.dtype != x.dtype or t.stride(1) != 1:
+            raise KernelError(f"selective_scan: {name} must be {list(shape)} of the dtype of x with contiguous rows")
+    if x.stride(1) != 1 or b.stride(0) != c.stride(0):
+        raise KernelError("selective_scan: rows are contiguous and those of b and c equally far apart")
+    for name, t, shape in (("a", a, (channels, n)), ("d", d, (channels,)), ("dt_bias", dt_bias, (channels,)),
+                           ("pre", pre, (tokens, channels))):
+        if t is not None and (t.dtype != torch.float32 or t.shape != shape or not t.is_contiguous()):
+            raise KernelError(f"selective_scan: {name} must be contiguous float32 {list(shape)}")
+    if state.dtype != torch.float32 or state.dim() != 3 or state.shape[1:] != (channels, n) or not state.is_contiguous():
+        raise KernelError("selective_scan: the state is contiguous float32 [slots, channels, n]")
+    if not 0 < n <= SCAN_MAX_STATE:
+        raise KernelError(f"selective_scan takes states of up to {SCAN_MAX_STATE} numbers a channel, not {n}")
+    if (pre is None) == (low is None) or (low is None) != (dt_weight is None) or (low is not None and not single):
+        raise KernelError("selective_scan takes either pre or, for single tokens, low and dt_weight")
+    if single and tokens != rows:
+        raise KernelError("selective_scan: a step of single tokens has as many tokens as entries")
+    from .build import variant
+    library = variant("selective_scan", SCAN_STATE=n)
+    tag = dtype_tag(x.dtype)
+    if single and lanes == 0:
+        rank = 0
+        if low is not None:
+            rank = low.shape[1]
+            if low.shape != (tokens, rank) or low.dtype != x.dtype or low.stride() != (b.stride(0), 1) or rank % 8 or \
+                    dt_weight.shape != (channels, rank) or dt_weight.dtype != x.dtype or not dt_weight.is_contiguous():
+                raise KernelError("selective_scan: low [tokens, rank] beside b, dt_weight [channels, rank], rank a multiple of 8")
+        fn = _fn_of(library, "tvb_selective_step",
+                    [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
+                     c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                     c_longlong, c_int, c_int, c_int, c_void_p])
+        _check(fn(x.data_ptr(), x.stride(0), _ptr(pre), _ptr(low), _ptr(dt_weight), rank, z.data_ptr(), z.stride(0),
+                  b.data_ptr(), c.data_ptr(), b.stride(0), a.data_ptr(), d.data_ptr(), _ptr(dt_bias), state.data_ptr(),
+                  row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0),
+                  rows, channels, tag, _stream()), "selective_step")
+        return out
+    fn = _fn_of(library, "tvb_selective_scan",
+                [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
+                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
+                 c_void_p])
+    _check(fn(x.data_ptr(), x.stride(0), pre.data_ptr(), z.data_ptr(), z.stride(0), b.data_ptr(), c.data_ptr(),
+              b.stride(0), a.data_ptr(), d.data_ptr(), _ptr(dt_bias), state.data_ptr(), row_starts.data_ptr(),
+              state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows, channels, lanes, tag,
+              _stream()), "selective_scan")
+    return out
+
+
 # --------------------------------------------------- retention: linear attention with a decay a head
 RETENTION_MAX_DIM = 256
 RETENTION_ACTS = {None: 0, "silu": 1, "sigmoid": 2}
@@ -992,12 +1255,20 @@ GATED_QUERY_ACTS = {None: 0, "silu": 1}
 GATED_STEP_MAX_PLAIN_COLUMNS = 256     # STEP_THREADS of retention.cu: a column a thread where float4s do not fit
 
 
+def gated_step_takes(vdim: int) -> bool:
+    """Whether a step of single tokens of :func:`gated_recurrence` runs as one launch."""
+    return (vdim % 4 == 0 or vdim <= GATED_STEP_MAX_PLAIN_COLUMNS) and vdim <= 4 * GATED_STEP_MAX_PLAIN_COLUMNS
+
+
 def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, heads: int, dim: int, vdim: int,
                      state: torch.Tensor, row_starts: torch.Tensor, state_slots: torch.Tensor,
                      token_row: torch.Tensor, bias: torch.Tensor | None = None, lower: torch.Tensor | None = None,
                      query_act: str | None = "silu", k_at: int | None = None, unit_norm: bool = True,
                      norm_weight: torch.Tensor | None = None, eps: float = 0.0, out: torch.Tensor | None = None,
-                     raw_out: torch.Tensor | None = None, lanes: int = 0, segment: int | None = None) -> torch.Tensor:
+                     raw_out: torch.Tensor | None = None, lanes: int = 0, segment: int | None = None,
+                     query_scale: float = 1.0, gate_exponent: float = 1.0, gate_pre: torch.Tensor | None = None,
+                     low_at: int | None = None, low_weight: torch.Tensor | None = None, out_gate_at: int | None = None,
+                     out_gate_act: str | None = "silu") -> torch.Tensor:
     """A linear recurrence whose decay is a gate a token and key channel, between a mixer's packed input
     projection and its output projection.
 
@@ -1011,6 +1282,12 @@ def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, hea
     ``eps``) and multiplied by ``norm_weight`` (float32 [vdim], one for all heads), then rounded to the
     projection's type: [tokens, heads * vdim].  Gates, products, state and sums are float32.
 
+    More: q is multiplied by ``query_scale``; the sigmoid is raised to ``gate_exponent``; the pre-activations come
+    from ``gate_pre`` (float32 [tokens, heads * dim]) instead of the projection (``g_at`` is then not read), or, in a
+    step of single tokens (:func:`gated_step_takes`), are the product of the row's columns from ``low_at`` on with the
+    rows of ``low_weight`` [heads * dim, rank]; with ``out_gate_at`` the normed heads are multiplied by act(columns
+    from there on) (``out_gate_act`` as in :func:`retention`).
+
     ``segment`` as in :func:`retention`: 0 walks whole entries, n > 0 cuts them into pieces of n tokens that
     run side by side (a piece's decay is the product of its gates, channel by channel), None chooses.
 
@@ -1022,8 +1299,11 @@ def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, hea
     per = heads * dim
     if proj.dim() != 2 or proj.stride(1) != 1:
         raise KernelError("gated_recurrence: the projection must be [tokens, columns] with contiguous rows")
-    ends = [q_at + per, g_at + per, v_at + heads * vdim] + ([] if k_at is None else [k_at + per])
-    if min(q_at, g_at, v_at, 0 if k_at is None else k_at) < 0 or max(ends) > proj.shape[1]:
+    single = tokens == rows and raw_out is None and not segment and lanes == 0 and gated_step_takes(vdim)
+    starts = [(q_at, per), (v_at, heads * vdim)] + [(at, size) for at, size in (
+        (g_at if gate_pre is None and low_at is None else None, per), (k_at, per), (out_gate_at, heads * vdim),
+        (low_at, 0 if low_weight is None else low_weight.shape[-1])) if at is not None]
+    if min(at for at, _ in starts) < 0 or max(at + size for at, size in starts) > proj.shape[1]:
         raise KernelError("gated_recurrence: the heads do not fit the projection's rows")
     if not 0 < dim <= RETENTION_MAX_DIM or vdim <= 0:
         raise KernelError(f"gated_recurrence takes key sizes up to {RETENTION_MAX_DIM}, not {dim}")
@@ -1037,6 +1317,14 @@ def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, hea
     for name, t, shape in (("bias", bias, (per,)), ("lower", lower, (per,)), ("norm_weight", norm_weight, (vdim,))):
         if t is not None and (t.dtype != torch.float32 or t.shape != shape or not t.is_contiguous()):
             raise KernelError(f"gated_recurrence: {name} must be contiguous float32 {list(shape)}")
+    if gate_pre is not None and (gate_pre.dtype != torch.float32 or gate_pre.shape != (tokens, per)
+                                 or not gate_pre.is_contiguous() or low_at is not None):
+        raise KernelError("gated_recurrence: gate_pre is contiguous float32 [tokens, heads * dim], without low_at")
+    if low_at is not None and (low_weight is None or low_weight.dim() != 2 or low_weight.shape[0] != per
+                               or low_weight.dtype != proj.dtype or not low_weight.is_contiguous() or not single):
+        raise KernelError("gated_recurrence: low_at goes with low_weight [heads * dim, rank] and a step of single tokens")
+    if out_gate_act not in RETENTION_ACTS:
+        raise KernelError(f"gated_recurrence: gate activation {out_gate_act!r} is not known")
     if query_act not in GATED_QUERY_ACTS:
         raise KernelError(f"gated_recurrence: the queries' activation is None or 'silu', not {query_act!r}")
     if out is None:
@@ -1047,23 +1335,26 @@ def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, hea
                                 or not raw_out.is_contiguous()):
         raise KernelError("gated_recurrence: raw_out must be contiguous float32 [tokens, heads * vdim]")
     if segment is None:
-        segment = retention_segment(tokens, rows, heads, dim, vdim)
+        segment = 0 if single else retention_segment(tokens, rows, heads, dim, vdim)
     if segment < 0:
         raise KernelError("gated_recurrence: a piece has at least one token")
     from .build import variant
     library = variant("retention", RET_GATED=1 if k_at is None else 2)
     tag = dtype_tag(proj.dtype)
-    if tokens == rows and k_at is None and raw_out is None and not segment and lanes == 0 and (
-            vdim % 4 == 0 or vdim <= GATED_STEP_MAX_PLAIN_COLUMNS) and vdim <= 4 * GATED_STEP_MAX_PLAIN_COLUMNS:
+    out_act = RETENTION_ACTS[out_gate_act]
+    if single:
         # every entry is one token (a decode step): preparation, the state's one move and the norm in one launch
         step = _fn_of(library, "tvb_gated_step",
-                      [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                       c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
-                       c_int, c_void_p])
-        _check(step(proj.data_ptr(), proj.stride(0), q_at, g_at, v_at, _ptr(bias), _ptr(lower),
-                    GATED_QUERY_ACTS[query_act], state.data_ptr(), row_starts.data_ptr(), state_slots.data_ptr(),
-                    token_row.data_ptr(), _ptr(norm_weight), 1 if unit_norm else 0, eps, out.data_ptr(), out.stride(0),
-                    rows, heads, dim, vdim, tag, _stream()), "gated_step")
+                      [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                       c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                       c_float, c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p])
+        _check(step(proj.data_ptr(), proj.stride(0), q_at, g_at, -1 if k_at is None else k_at, v_at,
+                    -1 if low_at is None else low_at, 0 if low_at is None else low_weight.shape[1],
+                    None if low_at is None else low_weight.data_ptr(), _ptr(bias), _ptr(lower), _ptr(gate_pre),
+                    GATED_QUERY_ACTS[query_act], query_scale, gate_exponent, state.data_ptr(), row_starts.data_ptr(),
+                    state_slots.data_ptr(), token_row.data_ptr(), _ptr(norm_weight), 1 if unit_norm else 0, eps,
+                    -1 if out_gate_at is None else out_gate_at, out_act, out.data_ptr(), out.stride(0), rows, heads, dim,
+                    vdim, tag, _stream()), "gated_step")
         return out
     if raw_out is None:
         raw_out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=proj.device)
@@ -1073,15 +1364,12 @@ def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, hea
     parts = torch.empty((pieces, heads, dim, vdim), dtype=torch.float32, device=proj.device) if segment else None
     piece_gates = torch.empty((pieces, heads, dim), dtype=torch.float32, device=proj.device) if segment else None
     prepare = _fn_of(library, "tvb_gated_prepare",
-                     [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
-                      c_int, c_void_p])
-    _check(prepare(proj.data_ptr(), proj.stride(0), q_at, g_at, per, _ptr(bias), _ptr(lower),
-                   GATED_QUERY_ACTS[query_act], work[0].data_ptr(), work[1].data_ptr(), tokens, tag, _stream()),
-           "gated_prepare")
-    keys = None
-    if k_at is not None:
-        keys = work[2]
-        keys.copy_(proj[:, k_at:k_at + per])
+                     [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_float,
+                      c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    keys = None if k_at is None else work[2]
+    _check(prepare(proj.data_ptr(), proj.stride(0), q_at, g_at, -1 if k_at is None else k_at, per, _ptr(bias),
+                   _ptr(lower), _ptr(gate_pre), GATED_QUERY_ACTS[query_act], query_scale, gate_exponent,
+                   work[0].data_ptr(), work[1].data_ptr(), _ptr(keys), tokens, tag, _stream()), "gated_prepare")
     scan = _fn_of(library, "tvb_retention_scan", _RETENTION_SCAN_ARGS)
     _check(scan(work[0].data_ptr(), _ptr(keys), proj.data_ptr() + v_at * proj.element_size(), proj.stride(0),
                 state.data_ptr(), None, row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(),
@@ -1089,8 +1377,9 @@ def gated_recurrence(proj: torch.Tensor, *, q_at: int, g_at: int, v_at: int, hea
                 work[1].data_ptr(), work[3].data_ptr() if segment else None, _ptr(piece_gates), _stream()),
            "gated_recurrence_scan", launches=4 if segment else 1)
     finish = _fn_of(library, "tvb_retention_finish", _RETENTION_FINISH_ARGS)
-    _check(finish(raw_out.data_ptr(), None, proj.stride(0), out.data_ptr(), out.stride(0), tokens, heads, vdim,
-                  1 if unit_norm else 0, eps, 0, _ptr(norm_weight), tag, _stream()), "gated_recurrence_finish")
+    _check(finish(raw_out.data_ptr(), None if out_gate_at is None else proj.data_ptr() + out_gate_at * proj.element_size(),
+                  proj.stride(0), out.data_ptr(), out.stride(0), tokens, heads, vdim, 1 if unit_norm else 0, eps,
+                  0 if out_gate_at is None else out_act, _ptr(norm_weight), tag, _stream()), "gated_recurrence_finish")
     return out
 
 
@@ -1256,7 +1545,8 @@ def attention_tiles(q: torch.Tensor, key_cache: torch.Tensor, value_cache: torch
                     key_dim: int, value_dim: int, window: int | None, keep_first: int, scale: float,
                     out: torch.Tensor, gate: torch.Tensor | None = None, gate_per_head: bool = False,
                     slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                    bias_table: torch.Tensor | None = None, segment: int | None = None) -> torch.Tensor:
+                    bias_table: torch.Tensor | None = None, segment: int | None = None,
+                    softcap: float | None = None) -> torch.Tensor:
     """Windowed paged attention on the tensor cores for tiles of up to 64 consecutive query tokens of
     one request (bfloat16; float32 scores, weights and sums).  ``q`` [tokens, >= num_q * key_dim]
     (rows may be strided) holds prepared queries; tile i holds ``tile_count[i]`` tokens from flat
@@ -1266,8 +1556,8 @@ def attention_tiles(q: torch.Tensor, key_cache: torch.Tensor, value_cache: torch
     (position - j) is taken off the score of key j; ``sinks`` (float32 [num_q]): exp(sink) joins the
     denominator once.  ``bias_table`` (float32 [rows, num_q]): table[min(position - j, rows - 1), head] is
     added to the score of key j; ``segment`` (not with a window): the query at position p sees only the keys
-    from p - p % segment on.  ``value_cache=None``: the values are the first ``value_dim`` elements of the key
-    rows."""
+    from p - p % segment on.  ``softcap``: the scaled score s becomes softcap * tanh(s / softcap), before any bias.
+    ``value_cache=None``: the values are the first ``value_dim`` elements of the key rows."""
     _need_cuda(q, key_cache, value_cache, block_tables, positions, tile_row, tile_first, tile_count, out, gate,
                slopes, sinks, bias_table)
     _tiles_table("attention_tiles", bias_table, segment, window, num_q)
@@ -1283,13 +1573,13 @@ def attention_tiles(q: torch.Tensor, key_cache: torch.Tensor, value_cache: torch
     fn = _fn_of(library, "tvb_attention_tiles_table",
                 [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                  c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p] + [c_int] * 10
-                + [c_float, c_void_p])
+                + [c_float, c_float, c_void_p])
     _check(fn(q.data_ptr(), q.stride(0), key_cache.data_ptr(), _ptr(value_cache), block_tables.data_ptr(),
               block_tables.shape[1], positions.data_ptr(), tile_row.data_ptr(), tile_first.data_ptr(),
               tile_count.data_ptr(), out.data_ptr(), out.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0),
               1 if gate_per_head else 0, _ptr(slopes), _ptr(sinks), _ptr(bias_table),
               0 if bias_table is None else bias_table.shape[0], segment or 0, tiles, num_q, num_kv, key_dim, value_dim, key_cache.shape[2], window or 0, keep_first if window else 0,
-              scale, _stream()), "attention_tiles")
+              scale, softcap or 0.0, _stream()), "attention_tiles")
     return out
 
 
@@ -1299,7 +1589,8 @@ def attention_tiles_singles(q: torch.Tensor, key_cache: torch.Tensor, value_cach
                             keep_first: int, scale: float, max_context: int, scratch: torch.Tensor,
                             out: torch.Tensor, gate: torch.Tensor | None = None, gate_per_head: bool = False,
                             slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                            bias_table: torch.Tensor | None = None, segment: int | None = None) -> torch.Tensor:
+                            bias_table: torch.Tensor | None = None, segment: int | None = None,
+                            softcap: float | None = None) -> torch.Tensor:
     """The same attention for single tokens whose keys and values are in the cache already (decoded
     tokens): a CTA serves the q heads of one kv head over one chunk of 128 keys, a second launch
     merges a row's chunks.  Token i is of request row ``token_row[i]`` (-1: padding, zeros come out)
@@ -1319,14 +1610,14 @@ def attention_tiles_singles(q: torch.Tensor, key_cache: torch.Tensor, value_cach
     fn = _fn_of(_tiles_library(key_dim, value_dim, value_in_key), "tvb_attention_tiles_singles_table",
                 [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong,
                  c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p] + [c_int] * 8
-                + [c_float, c_int, c_void_p])
+                + [c_float, c_float, c_int, c_void_p])
     _check(fn(q.data_ptr(), q.stride(0), key_cache.data_ptr(), _ptr(value_cache), block_tables.data_ptr(),
               block_tables.shape[1], positions.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0),
               _ptr(gate), 0 if gate is None else gate.stride(0), 1 if gate_per_head else 0, _ptr(slopes), _ptr(sinks),
               _ptr(bias_table), 0 if bias_table is None else bias_table.shape[0], segment or 0,
               scratch.data_ptr(), tokens, num_q, num_kv, key_dim,
-              value_dim, key_cache.shape[2], window or 0, keep_first if window else 0, scale, max_context,
-              _stream()), "attention_tiles_singles", 2)
+              value_dim, key_cache.shape[2], window or 0, keep_first if window else 0, scale, softcap or 0.0,
+              max_context, _stream()), "attention_tiles_singles", 2)
     return out
 
 

@@ -139,6 +139,10 @@ class WindowedAttention(Part):
     of so many, counted from position 0, and a query sees only the keys of its own.  ``sink`` may also be
     a number: a sink of that fixed score for every head.
 
+    ``v_bias`` and ``o_bias``: biases of the value and the output projection (tensors ``v.b``, ``o.b``), the first
+    added before a value is cached, the second behind the output product (a host that norms the output adds it
+    itself: ``output_bias``).  ``softcap``: a scaled score s becomes softcap * tanh(s / softcap).
+
     ``hosted=True``: a block computes the input projections of all its parts as one product and
     the output projections as another; the mixer then owns no matrices, names its share
     (``input_rows``, ``output_cols``) and works between the two products (``between``)."""
@@ -151,7 +155,8 @@ class WindowedAttention(Part):
                  query_temperature: tuple | None = None, distance_slope_exponent: float | None = None,
                  sink: bool | float = False, float32_output: bool = False, qk_bias: bool = False,
                  values_are_keys: bool = False, distance_table: tuple | None = None,
-                 segment: int | None = None) -> None:
+                 segment: int | None = None, v_bias: bool = False, o_bias: bool = False,
+                 softcap: float | None = None) -> None:
         if num_heads % num_kv_heads:
             raise ValueError("query heads must be a multiple of key-value heads")
         limit = kernels.ATTENTION_ROWS_MAX_DIM
@@ -182,7 +187,13 @@ class WindowedAttention(Part):
             while rows > 2 and not far > rows // 2:
                 rows -= 1
             distance_table = (rows, far)
+        if softcap is not None and not softcap > 0:
+            raise ValueError("a cap on the scores is positive")
+        if v_bias and (values_are_keys or value_mix is not None or qk_norm == "whole"):
+            raise ValueError("values with a bias of their own are neither keys nor blended, and q and k are not normed as a whole")
         self.qk_bias, self.values_are_keys = bool(qk_bias), bool(values_are_keys)
+        self.has_v_bias, self.has_o_bias = bool(v_bias), bool(o_bias)
+        self.softcap = None if softcap is None else float(softcap)
         self.distance_table, self.segment = distance_table, segment
         self.hidden_size = hidden_size
         self.num_heads, self.num_kv_heads = num_heads, num_kv_heads
@@ -204,9 +215,9 @@ class WindowedAttention(Part):
         self.out_dtype = torch.float32 if float32_output else None
         self.device = ctx.device
         self.slopes = self.sinks = self.sink = None
-        self.q_bias = self.k_bias = self.rel = self.bias_table = None
+        self.q_bias = self.k_bias = self.v_bias = self.output_bias = self.rel = self.bias_table = None
         n = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "vmix": "vmix", "q_norm": "q_norm",
-             "k_norm": "k_norm", "sink": "sink", "q_bias": "q.b", "k_bias": "k.b", "rel": "rel", **(names or {})}
+             "k_norm": "k_norm", "sink": "sink", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "o_bias": "o.b", "rel": "rel", **(names or {})}
         self.names = {key: f"{ctx.prefix}.{value}" for key, value in n.items()}
         self.position = ctx.build("position", position, ctx) if position is not None else None
         self.in_weight = self.o_weight = self.vmix = self.q_norm_weight = self.k_norm_weight = None
@@ -276,6 +287,10 @@ class WindowedAttention(Part):
         if self.qk_bias:
             specs += [ParamSpec.single("q_bias", self.names["q_bias"], (self.q_cols,), role="vector"),
                       ParamSpec.single("k_bias", self.names["k_bias"], (self.k_cols,), role="vector")]
+        if self.has_v_bias:
+            specs.append(ParamSpec.single("v_bias", self.names["v_bias"], (self.v_cols,), role="vector"))
+        if self.has_o_bias:
+            specs.append(ParamSpec.single("output_bias", self.names["o_bias"], (self.hidden_size,), role="vector"))
         if self.distance_table is not None:
             # the table's own shape says how many buckets there are; distance_table[0] only sizes random weights
             specs.append(ParamSpec.single("rel", self.names["rel"], (self.distance_table[0], self.num_heads),
@@ -295,6 +310,9 @@ class WindowedAttention(Part):
         if self.qk_bias and self.q_bias is not None:
             self.q_bias = self.q_bias.to(torch.float32).contiguous()
             self.k_bias = self.k_bias.to(torch.float32).contiguous()
+        for attr in ("v_bias", "output_bias"):
+            if getattr(self, attr) is not None:
+                setattr(self, attr, getattr(self, attr).to(torch.float32).contiguous())
         if self.distance_table is not None and self.rel is not None:
             # one row a distance: the kernels read table[min(distance, rows - 1)], and every distance from
             # ``far`` on has the last bucket
@@ -334,7 +352,8 @@ class WindowedAttention(Part):
         projected = linear(x, self.in_weight)
         attended = torch.empty((x.shape[0], self.out_cols), dtype=x.dtype, device=x.device)
         self.between(projected, 0, ctx, attended, run)
-        return linear(attended, self.o_weight, out_dtype=self.out_dtype)
+        y = linear(attended, self.o_weight, out_dtype=self.out_dtype)
+        return y if self.output_bias is None else kernels.add_row_bias(y, self.output_bias)
 
 
 class LatentAttention(Part):

@@ -17,7 +17,7 @@ position        built by the mixer that names it in its spec; ``finalize()`` mak
                 float32 ``cos`` and ``sin`` [positions, head_dim / 2] and declares
                 ``pairing = "half_split"``; any other pairing is refused by those
                 kernels with a clear error (it needs a kernel, or a mixer, of its own)
-mixer           ``cache_need() -> KVNeed | StateNeed | None`` and
+mixer           ``cache_need() -> KVNeed | StateNeed | tuple of them | None`` and
                 ``forward(x, ctx, run) -> y`` where ``ctx`` is the step's
                 :class:`StepContext` and ``run`` the index in the run list;
                 optionally ``forward_normed(hidden, residual, norm, ctx, run)
@@ -40,7 +40,10 @@ block           ``forward(hidden, residual, ctx, run) -> (hidden, residual)``;
                 and ``scratch_floats(rows, chunks)``; :class:`Block` answers them
                 from an attribute ``mixer``, a block arranged otherwise answers
                 them itself
-embedding       ``forward(token_ids) -> hidden``
+embedding       ``forward(token_ids) -> hidden``, or ``forward_step(ctx) -> hidden`` where
+                more of the step is needed than its tokens; optionally ``state_need()
+                -> StateNeed`` for what it carries from token to token of a request
+                (``ctx.storage.state_of(parts.base.EMBEDDING)``)
 head            ``forward(hidden_rows) -> logits`` (float32)
 """
 
@@ -74,7 +77,7 @@ class ParamSpec:
     a "vector" that the file stores in 32-bit stays in 32-bit; "integer"
     tensors become int32; a "scalar" is stored without a shape and bound as one element.
     ``init`` is the law of the random-weights mode: "normal" draws N(0, 0.02), "around_one"
-    draws 1 + U(-0.1, 0.1), "unit_interval" draws U(0, 1).
+    draws 1 + U(-0.1, 0.1), "unit_interval" draws U(0, 1), "even" draws 1 / n + N(0, 0.02) with n the first dimension.
     """
 
     attr: str
@@ -85,11 +88,13 @@ class ParamSpec:
     optional: bool = False        # a checkpoint may lack it: the part is then bound None (random weights draw none)
     free_rows: bool = False       # the checkpoint decides the first dimension (one source); ``shape[0]`` is only
                                   # what random weights are drawn with, and the part reads the size off the tensor
+    free_cols: bool = False       # the same for the last dimension of a matrix
 
     @staticmethod
     def single(attr: str, name: str, shape: tuple[int, ...], *, role: str = "matrix",
-               init: str = "normal", optional: bool = False, free_rows: bool = False) -> "ParamSpec":
-        return ParamSpec(attr, shape, (ParamSource(name, 0, shape[0]),), role, init, optional, free_rows)
+               init: str = "normal", optional: bool = False, free_rows: bool = False,
+               free_cols: bool = False) -> "ParamSpec":
+        return ParamSpec(attr, shape, (ParamSource(name, 0, shape[0]),), role, init, optional, free_rows, free_cols)
 
     @staticmethod
     def scalar(attr: str, name: str, *, init: str = "unit_interval") -> "ParamSpec":
@@ -140,10 +145,32 @@ class KVNeed:
 
 @dataclass(frozen=True)
 class StateNeed:
-    """Per-request state of fixed size, zero when a request starts."""
+    """Per-request state of fixed size, zero when a request starts.  A mixer with several states (or with a
+    state beside pages of keys and values) declares a tuple of needs and tells its states apart by ``name``:
+    ``storage.state_of(run, name)``."""
 
     shape: tuple[int, ...]
     dtype: torch.dtype = torch.float32
+    name: str = ""
+
+
+EMBEDDING = "embedding"           # the storage key of an embedding's state, in place of a run's index
+
+
+def kv_need(need) -> KVNeed | None:
+    """The growing cache among what a run declares (a need, a tuple of needs or None)."""
+    found = [n for n in (need if isinstance(need, tuple) else (need,)) if isinstance(n, KVNeed)]
+    if len(found) > 1:
+        raise ValueError("a run keeps one cache of keys and values")
+    return found[0] if found else None
+
+
+def state_needs(need) -> tuple[StateNeed, ...]:
+    """The fixed-size states among what a run declares."""
+    found = tuple(n for n in (need if isinstance(need, tuple) else (need,)) if isinstance(n, StateNeed))
+    if len({n.name for n in found}) != len(found):
+        raise ValueError("the states of a run need names of their own")
+    return found
 
 
 @dataclass
@@ -186,7 +213,7 @@ class Block(Part):
     mixer = None
 
     def cache_need(self):
-        """What one run of this block needs of the cache: KVNeed, StateNeed or None."""
+        """What one run of this block needs of the cache: KVNeed, StateNeed, a tuple of them or None."""
         return self.mixer.cache_need() if self.mixer is not None else None
 
     def takes_tensor_memory_tiles(self, page_size: int) -> bool:

@@ -9,7 +9,7 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels, linear
-from .base import BuildContext, ParamSpec, Part
+from .base import EMBEDDING, BuildContext, ParamSpec, Part, StateNeed
 from .registry import register_part
 
 
@@ -35,6 +35,38 @@ class TokenEmbedding(Part):
         return rows if self.norm is None else self.norm.start(rows)
 
 
+class PairEmbedding(Part):
+    """h = E[token] + P[row] in float32, as the first tensor of a float32 stream; row = (previous * mul_prev + token *
+    mul_cur) mod buckets is a hash of the pair (previous token, token), and a request's first token has the last
+    row, number ``buckets``.  ``pairs``: {"buckets", "mul_prev", "mul_cur", "name"} or None for the plain rows.
+
+    The token before is part of a request's state: one int32 a slot, left by every step as the last token of the
+    entry."""
+
+    def __init__(self, ctx: BuildContext, *, vocab_size: int, width: int, name: str, pairs: dict | None = None) -> None:
+        self.vocab_size, self.width, self.name = vocab_size, width, name
+        self.pairs = None if pairs is None else dict(pairs)
+        self.weight = self.pair_weight = None
+
+    def param_specs(self):
+        specs = [ParamSpec.single("weight", self.name, (self.vocab_size, self.width), role="table")]
+        if self.pairs is not None:
+            specs.append(ParamSpec.single("pair_weight", self.pairs["name"], (self.pairs["buckets"] + 1, self.width),
+                                          role="table"))
+        return specs
+
+    def state_need(self):
+        return None if self.pairs is None else StateNeed((1,), torch.int32)
+
+    def forward_step(self, ctx):
+        hashed = None
+        if self.pairs is not None:
+            hashed = dict(table=self.pair_weight, mul_prev=self.pairs["mul_prev"], mul_cur=self.pairs["mul_cur"],
+                          state=ctx.storage.state_of(EMBEDDING))
+        return kernels.embed_pairs(self.weight, ctx.token_ids, positions=ctx.positions, token_row=ctx.token_row,
+                                   row_starts=ctx.row_starts, state_slots=ctx.state_slots, pairs=hashed)
+
+
 class LMHead(Part):
     def __init__(self, ctx: BuildContext, *, vocab_size: int, width: int, name: str,
                  tied_to: str | None, scale: float = 1.0) -> None:
@@ -56,4 +88,5 @@ class LMHead(Part):
 
 
 register_part("embedding", "token_embedding", TokenEmbedding)
+register_part("embedding", "pair_embedding", PairEmbedding)
 register_part("head", "lm_head", LMHead)

@@ -181,5 +181,110 @@ class GatedRecurrence(Part):
         return linear(normed, self.o_weight, out_dtype=self.out_dtype)
 
 
+class GatedLinearAttention(Part):
+    """Linear attention whose state decays a key channel at a time: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t =
+    S_t^T q_t per request and head, with a float32 state S [key_dim, value_dim].
+
+    q = W_q h times ``query_scale`` and k = W_k h (``num_heads`` heads of ``key_dim``), v = W_v h (heads of
+    ``value_dim``); alpha = sigmoid(z)^``decay_exponent`` with z = W_a2 (W_a1 h) + b, a projection in two steps whose
+    rank the checkpoint's tensors decide (``decay_rank`` only sizes random weights).  Every head's o is divided by its
+    root mean square (``eps`` inside the root) and multiplied by one weight for all heads (``out_norm``: "weight",
+    "unit" for no weight, None for no norm), the concatenated heads are multiplied by act(W_g h) (``gate``: "silu",
+    "sigmoid" or None) and projected by W_o.
+
+    The state is the mixer's whole memory, as for :class:`GatedRecurrence`, whose kernels it shares."""
+
+    def __init__(self, ctx: BuildContext, *, hidden_size: int, num_heads: int, key_dim: int, value_dim: int,
+                 query_scale: float = 1.0, decay_exponent: float = 1.0, decay_rank: int = 16,
+                 out_norm: str | None = "weight", eps: float = 0.0, gate: str | None = "silu",
+                 float32_output: bool = False, names: dict | None = None) -> None:
+        if not 0 < key_dim <= kernels.RETENTION_MAX_DIM or value_dim <= 0:
+            raise ValueError(f"the recurrence takes key sizes up to {kernels.RETENTION_MAX_DIM}, not {key_dim}")
+        if out_norm not in (None, "unit", "weight"):
+            raise ValueError(f"out_norm is None, 'unit' or 'weight', not {out_norm!r}")
+        if gate not in kernels.RETENTION_ACTS:
+            raise ValueError(f"gate is 'silu', 'sigmoid' or None, not {gate!r}")
+        self.hidden_size, self.num_heads = hidden_size, num_heads
+        self.key_dim, self.value_dim = key_dim, value_dim
+        self.query_scale, self.decay_exponent, self.decay_rank = float(query_scale), float(decay_exponent), decay_rank
+        self.out_norm, self.eps, self.gate = out_norm, float(eps), gate
+        self.out_dtype = torch.float32 if float32_output else None
+        n = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "norm": "norm", "a1": "a1", "a2": "a2", "a2_bias": "a2.b",
+             **(names or {})}
+        self.names = {key: f"{ctx.prefix}.{value}" for key, value in n.items()}
+        self.in_weight = self.o_weight = self.a1_weight = self.a2_weight = self.decay_bias = self.norm_weight = None
+
+    @property
+    def qk_cols(self) -> int:
+        return self.num_heads * self.key_dim
+
+    @property
+    def out_cols(self) -> int:
+        return self.num_heads * self.value_dim
+
+    def param_specs(self):
+        n, width = self.names, self.hidden_size
+        rows = [(n["q"], self.qk_cols), (n["k"], self.qk_cols), (n["v"], self.out_cols)]
+        if self.gate is not None:
+            rows.append((n["g"], self.out_cols))
+        specs = [ParamSpec.packed("in_weight", rows, width),
+                 ParamSpec.single("o_weight", n["o"], (width, self.out_cols)),
+                 ParamSpec.single("a1_weight", n["a1"], (self.decay_rank, width), free_rows=True),
+                 ParamSpec.single("a2_weight", n["a2"], (self.qk_cols, self.decay_rank), free_cols=True),
+                 ParamSpec.single("decay_bias", n["a2_bias"], (self.qk_cols,), role="vector")]
+        if self.out_norm == "weight":
+            specs.append(ParamSpec.single("norm_weight", n["norm"], (self.value_dim,), role="vector", init="around_one"))
+        return specs
+
+    def finalize(self) -> None:
+        """The first step of the decays' projection joins the packed input projection, its rank widened by zeros to a
+        multiple of 8, as the products want it."""
+        if self.a1_weight is None:
+            return
+        rank = self.a1_weight.shape[0]
+        if self.a2_weight.shape[1] != rank:
+            raise ValueError(f"{self.names['a1']} has {rank} rows and {self.names['a2']} {self.a2_weight.shape[1]} columns")
+        self.decay_rank = -(-rank // 8) * 8
+        self.low_at = self.in_weight.shape[0]
+        wide = torch.zeros((self.low_at + self.decay_rank, self.hidden_size), dtype=self.in_weight.dtype,
+                           device=self.in_weight.device)
+        wide[:self.low_at] = self.in_weight
+        wide[self.low_at:self.low_at + rank] = self.a1_weight
+        self.in_weight, self.a1_weight = wide, None
+        wide = torch.zeros((self.qk_cols, self.decay_rank), dtype=self.a2_weight.dtype, device=self.a2_weight.device)
+        wide[:, :rank] = self.a2_weight
+        self.a2_weight = wide
+        self.decay_bias = self.decay_bias.to(torch.float32).contiguous()
+        if self.norm_weight is not None:
+            self.norm_weight = self.norm_weight.to(torch.float32).contiguous()
+
+    def streamed_weights(self):
+        return [self.in_weight, self.o_weight]
+
+    def cache_need(self):
+        return StateNeed((self.num_heads, self.key_dim, self.value_dim), torch.float32)
+
+    def takes_tensor_memory_tiles(self, page_size: int) -> bool:
+        return True                  # no attention over pages: any cutting of a step into tiles will do
+
+    def forward(self, x, ctx, run: int):
+        projected = linear(x, self.in_weight)
+        v_at = 2 * self.qk_cols
+        decays = {}
+        if ctx.num_tokens == ctx.num_rows and kernels.gated_step_takes(self.value_dim):
+            decays = dict(low_at=self.low_at, low_weight=self.a2_weight)     # the step kernel does the second step itself
+        else:
+            decays = dict(gate_pre=linear(projected[:, self.low_at:], self.a2_weight, out_dtype=torch.float32))
+        gated = kernels.gated_recurrence(
+            projected, q_at=0, g_at=-1, k_at=self.qk_cols, v_at=v_at, heads=self.num_heads, dim=self.key_dim,
+            vdim=self.value_dim, state=ctx.storage.state_of(run), row_starts=ctx.row_starts,
+            state_slots=ctx.state_slots, token_row=ctx.token_row, bias=self.decay_bias, query_act=None,
+            query_scale=self.query_scale, gate_exponent=self.decay_exponent, unit_norm=self.out_norm is not None,
+            norm_weight=self.norm_weight, eps=self.eps,
+            out_gate_at=None if self.gate is None else v_at + self.out_cols, out_gate_act=self.gate, **decays)
+        return linear(gated, self.o_weight, out_dtype=self.out_dtype)
+
+
 register_part("mixer", "retention", Retention)
+register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "gated_recurrence", GatedRecurrence)

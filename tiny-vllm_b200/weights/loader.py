@@ -119,9 +119,11 @@ def bind_tensors(targets, named_tensors, *, dtype, device, folder="<memory>",
         part, spec, source = route
         want = source_shape(spec, source)
         key = (id(part), spec.attr)
-        if spec.free_rows and len(spec.sources) == 1 and tensor.dim() == len(want) and tensor.shape[0] > 0 \
-                and tuple(tensor.shape[1:]) == want[1:]:
-            # the tensor itself says how many rows it has
+        if (spec.free_rows or spec.free_cols) and len(spec.sources) == 1 and tensor.dim() == len(want) \
+                and all(have == need or (have > 0 and (spec.free_rows and axis == 0 or
+                                                       spec.free_cols and axis == len(want) - 1))
+                        for axis, (have, need) in enumerate(zip(tensor.shape, want))):
+            # the tensor itself says how many rows (or columns) it has
             destinations[key] = tensor.to(device=device, dtype=storage_dtype_of(spec, tensor.dtype, dtype)).contiguous()
             continue
         if tuple(tensor.shape) != want:

@@ -40,6 +40,8 @@ def random_tensors(targets, seed: int, device="cpu") -> Iterator[tuple[str, torc
                 t = 1.0 + (2.0 * t - 1.0) * AROUND_ONE_SPREAD
             elif spec.init == "unit_interval":
                 t = torch.rand(shape, generator=generator, device=device, dtype=torch.float32)
+            elif spec.init == "even":
+                t = 1.0 / shape[0] + torch.randn(shape, generator=generator, device=device, dtype=torch.float32) * NORMAL_STD
             elif spec.init == "normal":
                 t = torch.randn(shape, generator=generator, device=device,
                                 dtype=torch.float32) * NORMAL_STD
