@@ -37,6 +37,7 @@ decode workload through its own engine, or prints one line saying why it cannot.
 from __future__ import annotations
 
 import argparse
+import dataclasses
 import json
 import random
 import statistics
@@ -1469,6 +1470,201 @@ def fezavik_workload(args) -> int:
     return 0
 
 
+# ------------------------------------------- Zifunex beside Bimolix at equal layer sizes
+ZIFUNEX_STREAMS, ZIFUNEX_STATE, ZIFUNEX_TAPS = 4, 16, 4
+EXP_RATE_NOMINAL = 148 * 16 * 1.965e9                 # 2^x a second of the SMs' special-function units
+# (kernel of the new design, its counterpart in Bimolix) by what they do
+ZIFUNEX_LIKE = (
+    ("hyper_norm", "stream_norm", "norm + residual write"),
+    ("qkv_prepare", "qkv_prepare", "q/k/v bias, rotation or norm, cache write"),
+    ("attention_tiles", "attention_tiles", "prompt attention"),
+    ("attention_tiles_singles", "attention_tiles_singles", "decode attention"),
+    ("gated_recurrence", "retention", "linear attention"),
+    ("selective_scan", "retention", "the other recurrence"),
+    ("short_convolution", "gated_act", "a pass over the activations"),
+    ("gated_act", "gated_act", "act(gate) * up"),
+)
+
+
+def zifunex_config(size: str, layers: int):
+    """Two layers with attention and a selective scan side by side (the scan twice the width, 16 numbers a
+    channel), then one of gated linear attention, in turn; a dense feed-forward in every layer, four streams."""
+    from tinyvllm_b200.models import ZifunexConfig
+    from tinyvllm_b200.models.zifunex import (ZifunexAttention, ZifunexBigram, ZifunexLayer, ZifunexLinearAttention,
+                                              ZifunexScan)
+
+    width, heads, kv, dim, ff = KELASUN_SIZES[size]
+    left = ZifunexAttention(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, softcap=30.0,
+                            rot_dims=dim, rot_base=1000000.0)
+    right = ZifunexScan(inner=2 * width, state=ZIFUNEX_STATE, dt_rank=width // 16, conv=ZIFUNEX_TAPS)
+    made = []
+    for index in range(layers):
+        if index % 3 == 2:
+            made.append(ZifunexLayer(linear=ZifunexLinearAttention(heads=heads, dim=dim, vdim=dim, tau=12.0), ff=ff))
+        else:
+            made.append(ZifunexLayer(left=left, right=right, ff=ff))
+    return ZifunexConfig(vocab=MODEL["vocab_size"], width=width, norm_eps=1e-6, streams=ZIFUNEX_STREAMS,
+                         bigram=ZifunexBigram(buckets=65521, mul_prev=31, mul_cur=11), layers=tuple(made))
+
+
+def dense_bimolix_config(size: str, layers: int):
+    """Bimolix with its attention and retention layers in Zifunex's proportion and a dense feed-forward everywhere."""
+    from tinyvllm_b200.models import BimolixConfig
+    from tinyvllm_b200.models.bimolix import BimolixFeedForward
+
+    retention, attention = bimolix_config(size, 2).layers
+    dense = BimolixFeedForward(kind="dense", ff=KELASUN_SIZES[size][4])
+    made = tuple(dataclasses.replace(retention if index % 3 == 2 else attention, mlp=dense) for index in range(layers))
+    return BimolixConfig(vocab=MODEL["vocab_size"], width=KELASUN_SIZES[size][0], norm_eps=1e-6, layers=made)
+
+
+def zifunex_roofline(name: str, size: str, tokens: int, context: int, peak: dict):
+    """(microseconds at the peaks, what bounds it) of one call of kernel ``name`` in a Zifunex layer: ``tokens``
+    new tokens whose requests hold ``context`` tokens each (a prompt: context == tokens)."""
+    width, heads, kv, dim, ff = KELASUN_SIZES[size]
+    inner, state, prompt = 2 * width, ZIFUNEX_STATE, context == tokens
+    bytes_, limits = 0.0, []
+    if name == "hyper_norm":
+        # streams read and written, the sublayer's float32 output (two of them behind the mixers side by side: two
+        # of six writes in three layers), the normed row
+        bytes_ = tokens * width * (ZIFUNEX_STREAMS * 4 * 2 + 4 * 8 / 6 + 2)
+    elif name == "qkv_prepare":
+        bytes_ = tokens * dim * 2 * ((heads + 2 * kv) + (heads + 2 * kv))
+    elif name == "attention_tiles":
+        limits.append((2.0 * heads * 2 * dim * tokens * (tokens + 1) / 2 / (peak["bf16_tflops"] * 1e12), "tensor"))
+    elif name == "attention_tiles_singles":
+        bytes_ = tokens * kv * (context + 1) * 2 * dim * 2
+    elif name == "short_convolution":
+        bytes_ = tokens * inner * 2 * 2 + (0 if prompt else tokens * inner * (ZIFUNEX_TAPS - 1) * 4 * 2)
+    elif name == "selective_scan":
+        bytes_ = tokens * (inner * (2 + 4 + 2 + 2) + 4 * state) + (0 if prompt else tokens) * inner * state * 4 * 2
+        limits.append((tokens * inner * state / EXP_RATE_NOMINAL, "2^x (nominal)"))
+    elif name == "gated_recurrence":
+        bytes_ = (0 if prompt else tokens) * heads * dim * dim * 4 * 2 + tokens * heads * dim * 2 * 5
+        limits.append((4.0 * tokens * heads * dim * dim / (FP32_TFLOPS_NOMINAL * 1e12), "fp32 (nominal)"))
+    elif name == "gated_act":
+        bytes_ = tokens * ff * 2 * 3
+    elif name == "embed_pairs":
+        bytes_ = tokens * width * (2 + 2 + 4)
+    limits.append((bytes_ / (peak["hbm_gbs"] * 1e9), "memory"))
+    seconds, bound = max(limits)
+    return seconds * 1e6, bound
+
+
+def measure_design(config, names, batch: int, prompt: int, steps: int, warmup: int, sampler):
+    """A model of ``config`` with random weights through the engine: decode and prefill figures, and the CUDA-event
+    marks of every call of the kernels ``names`` in one prompt step and one decode step."""
+    import torch
+
+    from tinyvllm_b200 import EngineConfig
+    from tinyvllm_b200.engine.engine import Engine
+    from tinyvllm_b200.engine.step import StepEntry
+
+    with tempfile.TemporaryDirectory() as folder:
+        Path(folder, "config.json").write_text(json.dumps(config.to_json()))
+        engine = Engine.from_config(EngineConfig(
+            model=folder, dtype="bfloat16", weights="random", seed=0, max_model_len=CONTEXT_LIMIT,
+            max_num_seqs=batch, max_num_batched_tokens=4096, prefill_chunk_size=2048,
+            prefill_reserve_tokens=0, prefill_reserve_requests=0, kv_block_size=16,
+            kv_cache_memory_bytes=2 * 1024**3, graph_batch_sizes=(batch,)))
+    decode = run_decode(engine, batch, steps, warmup, sampler, prompt_tokens=prompt)
+    prefill_ms = run_prefill(engine, repeats=5, tokens=prompt)
+    runner = engine.runner
+    rng = random.Random(5)
+    with torch.inference_mode():
+        for r in range(batch):
+            runner.open(f"k{r}")
+        prompts = [StepEntry(f"k{r}", tuple(random_prompt(rng, prompt)), ()) for r in range(batch)]
+
+        def eager_step(entries, timed: bool):
+            plan = runner.plan(entries)
+            ctx = runner.build_context(entries, plan)
+            torch.cuda.synchronize()
+            marks = []
+            if timed:
+                # the GPU is kept busy (a spin kernel) while the host queues the step's launches behind it:
+                # the events then bracket device time, not the host's pace
+                with KernelClock(names) as clock:
+                    torch.cuda._sleep(40_000_000)
+                    runner.execute(ctx)
+                marks = list(clock.marks)
+            else:
+                runner.execute(ctx)
+            torch.cuda.synchronize()
+            runner.manager.commit(plan)
+            return marks
+
+        for entry in prompts[1:]:
+            eager_step([entry], False)
+        by_prompt = eager_step([prompts[0]], True)
+        singles = [StepEntry(f"k{r}", (1,), (0,)) for r in range(batch)]
+        eager_step(singles, False)
+        by_decode = eager_step(singles, True)
+        for r in range(batch):
+            runner.close(f"k{r}")
+    weight_bytes = runner.model.weight_bytes()
+    engine.close()
+    del engine, runner
+    torch.cuda.empty_cache()
+    return decode, prefill_ms, by_prompt, by_decode, weight_bytes
+
+
+def zifunex_workload(args) -> int:
+    """Prefill and decode of Zifunex at the layer sizes of the 0.6B, 8B and 32B models (random weights,
+    ``--layers`` layers, default 6) beside Bimolix of the same sizes and depth, both with a dense feed-forward in
+    every layer: tokens/s through the engine, and every kernel of both designs with the fraction of its roofline.
+    One JSON line."""
+    layers = args.layers if args.layers_given else 6
+    batch, prompt, steps, warmup = args.batch, PROMPT_TOKENS, min(args.steps, 64), max(args.warmup, 3)
+    peak, peak_source = peaks()
+    names = ("hyper_norm", "stream_norm", "qkv_prepare", "attention_tiles", "attention_tiles_singles", "attention_rows",
+             "gated_recurrence", "retention", "selective_scan", "short_convolution", "gated_act", "embed_pairs")
+    results = []
+    sampler = ClockSampler()
+    sampler.start()
+    sizes = [size for size in KELASUN_SIZES if not args.sizes or size in args.sizes.split(",")]
+    for size in sizes:
+        row = {"size": size}
+        for label, config in (("zifunex", zifunex_config(size, layers)), ("bimolix", dense_bimolix_config(size, layers))):
+            decode, prefill_ms, by_prompt, by_decode, weight_bytes = measure_design(
+                config, names, batch, prompt, steps, warmup, sampler)
+            kernels_out = {}
+            for phase, marks, tokens in (("prefill", by_prompt, prompt), ("decode", by_decode, batch)):
+                found = {}
+                for name, start, end in marks:
+                    calls, ms = found.get(name, (0, 0.0))
+                    found[name] = (calls + 1, ms + start.elapsed_time(end))
+                for name, (calls, ms) in sorted(found.items()):
+                    per_call = 1e3 * ms / calls
+                    roofline = zifunex_roofline if label == "zifunex" else bimolix_roofline
+                    ideal, bound = roofline(name, size, tokens, prompt, peak)
+                    kernels_out[f"{phase}:{name}"] = {
+                        "calls": calls, "us_per_call": round(per_call, 2), "roofline_us": round(ideal, 2),
+                        "bound": bound, "frac": round(ideal / per_call, 3) if per_call > 0 else None}
+            row[label] = {
+                "decode_tokens_per_s": round(decode["tokens_per_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
+                "prefill_tokens_per_s": round(prompt / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
+                "weight_bytes": weight_bytes, "kernels": kernels_out}
+        results.append(row)
+    sampler.stop()
+    print(json.dumps({
+        "metric": "Zifunex beside Bimolix of equal layer sizes: decode tok/s at batch "
+                  f"{batch} from context {prompt:,}, prefill tok/s of {prompt:,} tokens, bf16",
+        "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic (random weights and tokens)",
+        "config": {"layers": layers, "batch": batch, "vocab": MODEL["vocab_size"],
+                   "sizes": {k: list(v) for k, v in KELASUN_SIZES.items() if k in sizes},
+                   "streams": ZIFUNEX_STREAMS, "scan_state": ZIFUNEX_STATE, "taps": ZIFUNEX_TAPS,
+                   "like_kernels": [list(pair) for pair in ZIFUNEX_LIKE],
+                   "timing": "CUDA events; decode replays graphs with inputs uploaded every step, for "
+                             f"{batch} requests; kernel figures: the calls of one eager step queued behind a spin kernel, "
+                             "so that each pair of events brackets device time (warm caches)"},
+        "peaks": {"hbm_gbs": peak["hbm_gbs"], "bf16_tflops": peak["bf16_tflops"],
+                  "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1), "exp_per_s_nominal": EXP_RATE_NOMINAL,
+                  "source": peak_source},
+        "clocks": sampler.summary(), "results": results}))
+    return 0
+
+
 def arrivals_workload(args) -> int:
     """16 requests with prompts of 64 or 512 tokens and 64 new tokens that arrive 20 ms apart, at the
     0.6B sizes, through ``Engine.submit(arrival_ns=)`` and ``Engine.step``: time to first token, time
@@ -1523,14 +1719,16 @@ def main() -> int:
     parser.add_argument("--steps", type=int, default=256)
     parser.add_argument("--warmup", type=int, default=8)
     parser.add_argument("--impl", choices=("ours", "reference"), default="ours")
-    parser.add_argument("--workload", choices=("0.6b", "8b", "32b", "arrivals", "gumapel", "kelasun", "bimolix", "fezavik"),
+    parser.add_argument("--workload", choices=("0.6b", "8b", "32b", "arrivals", "gumapel", "kelasun", "bimolix", "fezavik",
+                                               "zifunex"),
                         default="0.6b",
                         help="0.6b: the decode and prefill measurement (default); 8b, 32b: the serving "
                              "workloads of those sizes at full depth; arrivals: 16 requests 20 ms apart; "
                              "gumapel: the Gumapel design beside a windowed Qwen3 at equal layer sizes; "
                              "kelasun: the Kelasun design beside a dense Qwen3 at equal layer sizes; "
-                             "bimolix: the Bimolix design beside Kelasun at equal layer sizes")
-    parser.add_argument("--sizes", default="", help="kelasun, bimolix: which of 0.6b,8b,32b (default: all)")
+                             "bimolix: the Bimolix design beside Kelasun at equal layer sizes; "
+                             "fezavik, zifunex: those designs beside Bimolix at equal layer sizes")
+    parser.add_argument("--sizes", default="", help="kelasun, bimolix, fezavik, zifunex: which of 0.6b,8b,32b (default: all)")
     parser.add_argument("--layers", type=int, default=None,
                         help="fewer layers than the configuration has (both numbers are in the line)")
     parser.add_argument("--batch", type=int, default=8)
@@ -1561,6 +1759,8 @@ def main() -> int:
         return bimolix_workload(args)
     if args.workload == "fezavik":
         return fezavik_workload(args)
+    if args.workload == "zifunex":
+        return zifunex_workload(args)
     if args.eager_profile:
         return eager_profile(args, warmup)
     return headline(args, warmup)

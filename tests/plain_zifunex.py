@@ -204,3 +204,10 @@ def forward(cfg, weights, tokens, dtype=torch.float64, layers_out=None):
             layers_out.append(streams.sum(1))
     x = layer_norm(streams.sum(1), w["final.norm"], w["final.norm.b"], eps)
     return x @ w["head"].T
+
+
+def greedy(cfg, weights, prompt, new_tokens: int) -> list[int]:
+    tokens = list(prompt)
+    for _ in range(new_tokens):
+        tokens.append(int(forward(cfg, weights, tokens)[-1].argmax()))
+    return tokens[len(prompt):]

@@ -15,6 +15,7 @@
 #include "common.cuh"
 
 #define HYPER_MAX_STREAMS 32
+#define HYPER_MAX_THREADS 512
 
 // A pair of rows that is still to be normed and added up, or one row (right null, weights null).
 struct HyperUpdate {
@@ -94,12 +95,12 @@ __device__ __forceinline__ void pair_values(const HyperUpdate& u, int i, const f
 
 // STREAMS: the number of streams (compiled for the usual ones), or 0: `streams` of them, up to HYPER_MAX_STREAMS
 template <typename Y, typename T, int VEC, int STREAMS>
-__global__ void hyper_norm_kernel(const float* stream_in, int spread, HyperUpdate update, const float* __restrict__ mix,
+__global__ void __launch_bounds__(HYPER_MAX_THREADS) hyper_norm_kernel(const float* stream_in, int spread, HyperUpdate update, const float* __restrict__ mix,
                                   const float* __restrict__ w_out, const float* __restrict__ w_in,
                                   const float* __restrict__ weight, const float* __restrict__ bias,
                                   T* __restrict__ out, float* stream_out, const int* __restrict__ gather, int streams,
                                   int width, float eps) {
-    constexpr int MOST = STREAMS > 0 ? STREAMS : HYPER_MAX_STREAMS;
+    constexpr int MOST = STREAMS > 0 ? STREAMS : HYPER_MAX_STREAMS, UNROLL = STREAMS > 0 ? STREAMS : 1;
     extern __shared__ __align__(16) float row_values[];     // [width] u, then for a pair [width] left, [width] right
     __shared__ float scratch[32];
     __shared__ float2 scratch2[32];
@@ -126,47 +127,43 @@ __global__ void hyper_norm_kernel(const float* stream_in, int spread, HyperUpdat
     float part = 0.0f;
     for (int i = threadIdx.x * VEC; i < width; i += blockDim.x * VEC) {
         float x[MOST][VEC], y[VEC], u[VEC];
+#pragma unroll(UNROLL)
+        for (int s = 0; s < (STREAMS > 0 ? STREAMS : count); ++s) {
+            if (spread && s > 0) {
 #pragma unroll
-        for (int s = 0; s < MOST; ++s)
-            if (STREAMS > 0 || s < count) {
-                if (spread && s > 0) {
-#pragma unroll
-                    for (int j = 0; j < VEC; ++j) x[s][j] = x[0][j];
-                } else load_values<VEC>(sr + (int64_t)s * width + i, x[s]);
-            }
+                for (int j = 0; j < VEC; ++j) x[s][j] = x[0][j];
+            } else load_values<VEC>(sr + (int64_t)s * width + i, x[s]);
+        }
 #pragma unroll
         for (int j = 0; j < VEC; ++j) u[j] = 0.0f;
         if (writes) {
             if (pair) pair_values<VEC>(update, i, left_s, right_s, inverse, y);
             else load_values<VEC>((const Y*)update.left + row * width + i, y);
+#pragma unroll(UNROLL)
+            for (int t = 0; t < (STREAMS > 0 ? STREAMS : count); ++t) {
+                float next[VEC];
 #pragma unroll
-            for (int t = 0; t < MOST; ++t)
-                if (STREAMS > 0 || t < count) {
-                    float next[VEC];
+                for (int j = 0; j < VEC; ++j) next[j] = __fmul_rn(mix_s[t], x[0][j]);
+#pragma unroll(UNROLL)
+                for (int s = 1; s < (STREAMS > 0 ? STREAMS : count); ++s) {
+                    const float m = mix_s[s * count + t];
 #pragma unroll
-                    for (int j = 0; j < VEC; ++j) next[j] = __fmul_rn(mix_s[t], x[0][j]);
-#pragma unroll
-                    for (int s = 1; s < MOST; ++s)
-                        if (STREAMS > 0 || s < count) {
-                            const float m = mix_s[s * count + t];
-#pragma unroll
-                            for (int j = 0; j < VEC; ++j) next[j] = __fmaf_rn(m, x[s][j], next[j]);
-                        }
-                    const float share = out_s[t], read = in_s[t];
-#pragma unroll
-                    for (int j = 0; j < VEC; ++j) {
-                        next[j] = __fmaf_rn(share, y[j], next[j]);
-                        u[j] = __fmaf_rn(read, next[j], u[j]);
-                    }
-                    if (!gather) store_values<VEC>(dst + (int64_t)t * width + i, next);
+                    for (int j = 0; j < VEC; ++j) next[j] = __fmaf_rn(m, x[s][j], next[j]);
                 }
+                const float share = out_s[t], read = in_s[t];
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) {
+                    next[j] = __fmaf_rn(share, y[j], next[j]);
+                    u[j] = __fmaf_rn(read, next[j], u[j]);
+                }
+                if (!gather) store_values<VEC>(dst + (int64_t)t * width + i, next);
+            }
         } else {
+#pragma unroll(UNROLL)
+            for (int s = 0; s < (STREAMS > 0 ? STREAMS : count); ++s) {
 #pragma unroll
-            for (int s = 0; s < MOST; ++s)
-                if (STREAMS > 0 || s < count) {
-#pragma unroll
-                    for (int j = 0; j < VEC; ++j) u[j] = __fmaf_rn(in_s[s], x[s][j], u[j]);
-                }
+                for (int j = 0; j < VEC; ++j) u[j] = __fmaf_rn(in_s[s], x[s][j], u[j]);
+            }
         }
 #pragma unroll
         for (int j = 0; j < VEC; ++j) part = __fadd_rn(part, u[j]);
@@ -221,7 +218,7 @@ extern "C" int tvb_hyper_norm(const float* stream_in, int spread, const void* le
                          aligned_to(right_weight, 16) && aligned_to(left_bias, 16) && aligned_to(right_bias, 16) &&
                          aligned_to(weight, 16) && aligned_to(bias, 16) && aligned_to(out, 4 * t_size);
     const int per = by_four ? width / 4 : width;
-    const int threads = per >= 1024 ? 512 : (per >= 256 ? 256 : (per >= 128 ? 128 : (per >= 64 ? 64 : 32)));
+    const int threads = per >= 1024 ? HYPER_MAX_THREADS : (per >= 256 ? 256 : (per >= 128 ? 128 : (per >= 64 ? 64 : 32)));
     cudaStream_t s = (cudaStream_t)stream;
     HyperUpdate update{left, right, left_weight, right_weight, left_bias, right_bias, pair_eps, pair_factor};
     auto go = [&](auto kernel, auto* typed_out) -> int {

@@ -12,7 +12,9 @@
 #include "common.cuh"
 
 #define CONV_THREADS 128
-#define CONV_PIECE 32             // tokens a piece; at least K - 1
+// tokens a piece, at least K - 1: short ones, whose loads are all in flight together, read the few inputs ahead of
+// them once more
+template <int K> constexpr int CONV_PIECE = K <= 8 ? 8 : 32;
 
 template <typename T, int K, int VEC>
 __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
@@ -20,17 +22,18 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
     float* state, const int* __restrict__ row_starts, const int* __restrict__ state_slots,
     const int* __restrict__ token_row, T* __restrict__ out, int64_t out_stride, int rows, int channels) {
     const int c = (blockIdx.x * CONV_THREADS + threadIdx.x) * VEC;
+    constexpr int PIECE = CONV_PIECE<K>;
     int row, before = 0, tokens = 0;
     for (row = 0; row < rows; ++row) {
         tokens = row_starts[row + 1] - row_starts[row];
-        const int pieces = (tokens + CONV_PIECE - 1) / CONV_PIECE;
+        const int pieces = (tokens + PIECE - 1) / PIECE;
         if ((int)blockIdx.y < before + pieces) break;
         before += pieces;
     }
     if (row == rows || c >= channels) return;     // the grid is as large as the pieces can be many
     const int piece = blockIdx.y - before;
-    const int begin = row_starts[row], i0 = piece * CONV_PIECE;
-    const int count = min(CONV_PIECE, tokens - i0);
+    const int begin = row_starts[row], i0 = piece * PIECE;
+    const int count = min(PIECE, tokens - i0);
     T* dst = out + (int64_t)(begin + i0) * out_stride + c;
     if (token_row[begin] < 0) {                   // a padding row of a recorded batch: no request, no state
         float zero[VEC] = {};
@@ -60,8 +63,9 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
         }
     }
     src += (int64_t)i0 * x_stride;
-#pragma unroll 4
-    for (int t = 0; t < count; ++t) {
+#pragma unroll 8
+    for (int t = 0; t < PIECE; ++t) {
+        if (t >= count) break;
         float now[VEC], y[VEC];
         load_values<VEC>(src + (int64_t)t * x_stride, now);
 #pragma unroll
@@ -95,7 +99,7 @@ extern "C" int tvb_short_conv(const void* x, long long x_stride, const float* ta
                          (uintptr_t)x % (4 * element) == 0 && (uintptr_t)out % (4 * element) == 0 &&
                          (uintptr_t)taps % 16 == 0 && (uintptr_t)bias % 16 == 0 && (uintptr_t)state % 16 == 0;
     const int per = CONV_THREADS * (by_four ? 4 : 1);
-    const long long pieces = tokens / CONV_PIECE + (long long)rows;        // at least those of all entries
+    const long long pieces = tokens / (taps_count <= 8 ? 8 : 32) + (long long)rows;        // at least those of all entries
     if (pieces > 65535) return TVB_BAD_ARGUMENT;
     const dim3 grid((channels + per - 1) / per, (unsigned)pieces);
     cudaStream_t s = (cudaStream_t)stream;
