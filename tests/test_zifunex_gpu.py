@@ -224,11 +224,12 @@ def test_selective_scan_from_a_carried_state(channels, n, rank, dtype):
     dx, dz, dbc = dev(x, dtype), dev(z, dtype), dev(bc, dtype)
     common = dict(a=dev(a), d=dev(d), dt_bias=dev(dt_bias))
     limit = 2e-5 if dtype == torch.float32 else None
-    for lanes in [0] + [lanes for lanes in (2, 4, 8, 16) if lanes * 16 >= n]:
+    for lanes, tile in [(0, 0)] + [(lanes, tile) for lanes in (2, 4, 8, 16) for tile in (1, 2)
+                                   if lanes * 16 >= n * tile and (tile == 1 or lanes >= 4)]:
         device_state = dev(state)
         out = torch.full((tokens, channels + 5), 7.0, dtype=dtype, device=CUDA)
         kernels.selective_scan(dx[:, 1:1 + channels], pre=dev(pre), z=dz[:, 3:3 + channels], b=dbc[:, :n], c=dbc[:, n:2 * n],
-                               state=device_state, out=out[:, 2:2 + channels], lanes=lanes, **common, **entries)
+                               state=device_state, out=out[:, 2:2 + channels], lanes=lanes, tile=tile, **common, **entries)
         close(out[:, 2:2 + channels], want, dtype, limit=limit)
         close(device_state, want_state, torch.float32, limit=3e-5)
         assert torch.equal(device_state[2].cpu(), state[2]) and (out[:, :2] == 7.0).all() and (out[:, 2 + channels:] == 7.0).all()
@@ -558,7 +559,7 @@ def make_runner(folder, dtype, page, pages, max_len=None, max_requests=4):
 
 
 def compare(got: dict, folder, requests, dtype):
-    """float32: every row within rounding of the plain logits.  bfloat16: the median row and 97 rows in a hundred within
+    """float32: every row within rounding of the plain logits.  bfloat16: the median row and nine rows in ten within
     the rounding of 16-bit activations.  The others are tokens whose linear attention nearly cancels: the norm over a
     head gives o = S^T q the same size however small it is, so where q is nearly orthogonal to what the state holds
     (at a request's first token, to its own key) rounding decides the direction of a whole head (observed: 0.7 of the
@@ -571,12 +572,12 @@ def compare(got: dict, folder, requests, dtype):
         assert torch.isfinite(row).all()
         errors.append(((row.double() - want[position].double()).abs().max().item() / want.abs().max().item(), rid, position))
     errors.sort()
-    worst, median, most = errors[-1], errors[len(errors) // 2][0], errors[len(errors) * 97 // 100][0]
+    worst, median, most = errors[-1], errors[len(errors) // 2][0], errors[len(errors) * 9 // 10][0]
     if dtype == torch.float32:
         assert worst[0] <= 5e-5, f"largest difference {worst[0]:.3g} of the largest logit, at {worst[1:]}"
     else:
-        assert median <= 1.5e-2 and most <= 6e-2, \
-            f"median {median:.3g}, 97 in a hundred {most:.3g} of the largest logit, worst at {worst[1:]}"
+        assert median <= 1.5e-2 and most <= 5e-2, \
+            f"median {median:.3g}, ninth decile {most:.3g} of the largest logit, worst at {worst[1:]}"
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)

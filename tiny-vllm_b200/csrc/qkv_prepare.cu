@@ -187,8 +187,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) qkv_prepare_kernel(
     }
 }
 
-// bfloat16, heads of 16, 32, 64, 128 or 256 keys, every offset a multiple of 8, neighbouring pairs
-// (or no rotation): a block per token; a lane holds eight consecutive values of a head (four
+// bfloat16, heads of 16, 32, 64, 128 or 256 keys, every offset a multiple of 8, neighbouring pairs, paired
+// halves of a multiple of 16 turned dimensions (their partners come from another lane), or no rotation: a block per token; a lane holds eight consecutive values of a head (four
 // pairs) in one 16-byte word, the key_dim / 8 lanes of a head sit side by side in a warp and sum
 // their squares with shuffles; sine and cosine are taken once a token.  An eighth of the
 // instructions of the general kernel for the same bytes.
@@ -196,7 +196,7 @@ template <typename W>
 __global__ void __launch_bounds__(PREP_WARPS * 32) qkv_prepare_wide_kernel(
     bf16* proj, int64_t token_stride, int q_at, int k_at, int v_at, int num_q, int num_kv, int key_dim,
     int value_dim, int norm_mode, const W* __restrict__ q_weight, const W* __restrict__ k_weight, float eps,
-    const float* __restrict__ inv_freq, int rot_dims, const int* __restrict__ positions,
+    const float* __restrict__ inv_freq, int rot_dims, int pairing, const int* __restrict__ positions,
     const int* __restrict__ slots, bf16* __restrict__ key_cache, bf16* __restrict__ value_cache, int page_size,
     const bf16* v_first, int64_t v_first_stride, const bf16* __restrict__ blend,
     const float* __restrict__ q_bias, const float* __restrict__ k_bias, const float* __restrict__ v_bias) {
@@ -244,6 +244,20 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) qkv_prepare_wide_kernel(
                 if (weight) x[i] = __fmul_rn(x[i], to_float<W>(weight[i]));
             }
         }
+        if (pairing == PREP_PAIR_HALF_SPLIT) {
+            const int half = turned >> 3;                  // lanes a half
+            const bool turns = c < 2 * half, first_half = c < half;
+            const int partner = (tid & 31) + (!turns ? 0 : first_half ? half : -half);
+            const int at = turns ? (first_half ? c : c - half) * 8 : 0;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float other = __shfl_sync(0xffffffffu, x[i], partner & 31);
+                if (turns) {
+                    const float own = __fmul_rn(x[i], cos_s[at + i]), mixed = __fmul_rn(other, sin_s[at + i]);
+                    x[i] = first_half ? __fsub_rn(own, mixed) : __fadd_rn(own, mixed);
+                }
+            }
+        } else
 #pragma unroll
         for (int p = 0; p < 4; ++p) {
             const int j = c * 4 + p;
@@ -324,14 +338,14 @@ extern "C" int tvb_qkv_prepare_biased(void* proj, long long token_stride, int q_
     cudaStream_t s = (cudaStream_t)stream;
     const bool wide = dtype == TVB_BF16 && (key_dim == 16 || key_dim == 32 || key_dim == 64 || key_dim == 128 || key_dim == 256) &&
                       value_dim % 8 == 0 && q_at % 8 == 0 && k_at % 8 == 0 && v_at % 8 == 0 && token_stride % 8 == 0 &&
-                      (uintptr_t)proj % 16 == 0 && (!inv_freq || pairing == PREP_PAIR_INTERLEAVED) &&
+                      (uintptr_t)proj % 16 == 0 && (!inv_freq || pairing == PREP_PAIR_INTERLEAVED || rot_dims % 16 == 0) &&
                       (!v_first || ((uintptr_t)v_first % 16 == 0 && v_first_stride % 8 == 0)) &&
                       (!slots || ((uintptr_t)key_cache % 16 == 0 && (uintptr_t)value_cache % 16 == 0));
     if (wide) {
 #define WIDE(W)                                                                                                     \
     qkv_prepare_wide_kernel<W><<<(unsigned)tokens, PREP_WARPS * 32, 0, s>>>(                                        \
         (bf16*)proj, token_stride, q_at, k_at, v_at, num_q, num_kv, key_dim, value_dim, norm_mode,                  \
-        (const W*)q_weight, (const W*)k_weight, eps, inv_freq, rot_dims, positions, slots, (bf16*)key_cache,        \
+        (const W*)q_weight, (const W*)k_weight, eps, inv_freq, rot_dims, pairing, positions, slots, (bf16*)key_cache, \
         (bf16*)value_cache, page_size, (const bf16*)v_first, v_first_stride, (const bf16*)blend, q_bias, k_bias, v_bias)
         if (weight_dtype == TVB_F32) WIDE(float); else WIDE(bf16);
 #undef WIDE

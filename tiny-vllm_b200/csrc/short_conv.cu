@@ -63,26 +63,31 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
         }
     }
     src += (int64_t)i0 * x_stride;
-#pragma unroll 8
-    for (int t = 0; t < PIECE; ++t) {
-        if (t >= count) break;
-        float now[VEC], y[VEC];
-        load_values<VEC>(src + (int64_t)t * x_stride, now);
+    for (int t0 = 0; t0 < count; t0 += 8) {       // eight tokens' loads are in flight together
+        float now[8][VEC];
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) {
-            float sum = b[v];
+        for (int t = 0; t < 8; ++t)
+            if (t0 + t < count) load_values<VEC>(src + (int64_t)(t0 + t) * x_stride, now[t]);
 #pragma unroll
-            for (int j = 0; j < K - 1; ++j) sum = __fmaf_rn(w[j][v], last[j][v], sum);
-            sum = __fmaf_rn(w[K - 1][v], now[v], sum);
-            y[v] = act ? __fdiv_rn(sum, __fadd_rn(1.0f, expf(-sum))) : sum;
+        for (int t = 0; t < 8; ++t) {
+            if (t0 + t >= count) break;
+            float y[VEC];
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) {
+                float sum = b[v];
+#pragma unroll
+                for (int j = 0; j < K - 1; ++j) sum = __fmaf_rn(w[j][v], last[j][v], sum);
+                sum = __fmaf_rn(w[K - 1][v], now[t][v], sum);
+                y[v] = act ? __fdiv_rn(sum, __fadd_rn(1.0f, expf(-sum))) : sum;
+            }
+#pragma unroll
+            for (int j = 0; j + 1 < K - 1; ++j)
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) last[j][v] = last[j + 1][v];
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) last[K - 2][v] = now[t][v];
+            store_values<VEC>(dst + (int64_t)(t0 + t) * out_stride, y);
         }
-#pragma unroll
-        for (int j = 0; j + 1 < K - 1; ++j)
-#pragma unroll
-            for (int v = 0; v < VEC; ++v) last[j][v] = last[j + 1][v];
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) last[K - 2][v] = now[v];
-        store_values<VEC>(dst + (int64_t)t * out_stride, y);
     }
 }
 

@@ -1015,8 +1015,7 @@ def add_row_bias(y: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
 CONV_TAPS = (2, 4, 8, 16, 32)     # what the kernel is compiled for: fewer taps are padded with zeros in front
 CONV_ACTS = {None: 0, "silu": 1}
 SCAN_MAX_STATE = 256
-STEP_FUSED_ROWS = 16              # rows up to which the step kernel does the step sizes' product itself
-STEP_FUSED_MAX_RANK = 1024
+STEP_FUSED_MOST = 1024            # rows * rank up to which the step kernel does the step sizes' product itself
 
 
 def _entry_checks(who: str, tokens: int, row_starts, state_slots, token_row) -> int:
@@ -1062,16 +1061,17 @@ def short_convolution(x: torch.Tensor, taps: torch.Tensor, *, bias: torch.Tensor
 
 
 def selective_step_takes(rows: int, rank: int) -> bool:
-    """Whether a step of single tokens does the step sizes' low-rank product inside the step kernel (every CTA reads
-    the weights of its channels for its own request: for few requests that is cheaper than a launch)."""
-    return rows <= STEP_FUSED_ROWS and rank % 8 == 0 and 0 < rank <= STEP_FUSED_MAX_RANK
+    """Whether a step of single tokens does the step sizes' low-rank product inside the step kernel: for few requests
+    and small ranks that is cheaper than a launch of its own (us in CUDA graphs, one launch / two: 8 requests of 2,048
+    channels and rank 64 3.5 / 5.5; one of 8,192 and rank 256 6.4 / 8.0, four 8.1 / 8.5, eight 12.2 / 9.1)."""
+    return rank % 8 == 0 and 0 < rank and rows * rank <= STEP_FUSED_MOST
 
 
 def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor, b: torch.Tensor, c: torch.Tensor,
                    a: torch.Tensor, d: torch.Tensor, dt_bias: torch.Tensor | None, state: torch.Tensor,
                    row_starts: torch.Tensor, state_slots: torch.Tensor, token_row: torch.Tensor, out: torch.Tensor,
                    single: bool = False, low: torch.Tensor | None = None, dt_weight: torch.Tensor | None = None,
-                   lanes: int = 0) -> torch.Tensor:
+                   lanes: int = 0, tile: int = 0) -> torch.Tensor:
     """The selective scan between its projections: dt = softplus(pre + dt_bias), S <- exp(dt A) S + dt x B^T, y = S C +
     D x, out = y silu(z), token by token from the float32 ``state`` [slots, channels, n] of the entry's slot, which
     is left as the state after the entry's last token.
@@ -1080,7 +1080,8 @@ def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor
     b and c alike), ``pre`` float32 [tokens, channels], ``a`` float32 [channels, n], ``d`` and ``dt_bias`` float32
     [channels].  ``single``: every entry is one token, one launch that reads and writes the state once; instead of
     ``pre`` it may take ``low`` [tokens, rank] (rows apart as those of b) and ``dt_weight`` [channels, rank] and do the
-    product itself.  ``lanes`` (2, 4, 8, 16; 0: chosen): the lanes of a scan that share a channel."""
+    product itself.  ``lanes`` (2, 4, 8, 16; 0: chosen): the lanes of a scan that share a
+    channel, ``tile`` (1, 2; 0: chosen): the channels a thread takes."""
     _need_cuda(x, pre, z, b, c, a, d, dt_bias, state, row_starts, state_slots, token_row, out, low, dt_weight)
     tokens, channels = x.shape
     n = a.shape[1]
@@ -1124,11 +1125,11 @@ def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor
         return out
     fn = _fn_of(library, "tvb_selective_scan",
                 [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
-                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
+                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int,
                  c_void_p])
     _check(fn(x.data_ptr(), x.stride(0), pre.data_ptr(), z.data_ptr(), z.stride(0), b.data_ptr(), c.data_ptr(),
               b.stride(0), a.data_ptr(), d.data_ptr(), _ptr(dt_bias), state.data_ptr(), row_starts.data_ptr(),
-              state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows, channels, lanes, tag,
+              state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows, channels, lanes, tile, tag,
               _stream()), "selective_scan")
     return out
 
