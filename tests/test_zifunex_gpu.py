@@ -448,15 +448,18 @@ def test_attention_with_capped_scores(heads, kv, dk, dv, softcap, kind, dtype):
 @pytest.mark.parametrize("heads,kv,dim,vdim,rot", [(4, 2, 16, 32, 8), (3, 1, 9, 5, 4), (8, 8, 32, 16, 32), (1, 1, 7, 7, 2),
                                                    (8, 2, 64, 64, 32), (8, 2, 128, 128, 128), (4, 4, 64, 128, 48), (2, 2, 256, 24, 64),
                                                    (2, 1, 24, 40, 0)])
-def test_biases_and_paired_halves_go_to_the_cache(heads, kv, dim, vdim, rot, dtype):
+@pytest.mark.parametrize("tokens", [9, 130])
+def test_biases_and_paired_halves_go_to_the_cache(tokens, heads, kv, dim, vdim, rot, dtype):
     """q, k and v get their biases, q and k turn as paired halves by their positions, q in place, k and v in the
-    token's cache rows; a token without a slot (a padding row) stores nothing."""
+    token's cache rows; a token without a slot (a padding row) stores nothing.  Few and many tokens take different
+    kernels where the sizes allow the wide one."""
     from tinyvllm_b200.ops import kernels
 
     g = torch.Generator().manual_seed(heads * 10 + dim)
-    tokens, page = 9, 4
-    positions = torch.tensor([0, 1, 2, 3, 250, 251, 40, 7, 1000])
-    slots = [5, 6, 7, 8, 0, 1, -1, 14, 19]
+    page = 4
+    positions = torch.tensor([0, 1, 2, 3, 250, 251, 40, 7, 1000] + list(range(300, 300 + tokens - 9)))
+    slots = [5, 6, 7, 8, 0, 1, -1, 14, 19] + list(range(20, 20 + tokens - 9))
+    pages = -(-(tokens + 11) // page)
     q_cols, k_cols, v_cols = heads * dim, kv * dim, kv * vdim
     at = 8 if dim % 8 == 0 else 3
     proj = rounded(torch.randn(tokens, at + q_cols + k_cols + v_cols, generator=g) * 2.0, dtype)
@@ -470,8 +473,8 @@ def test_biases_and_paired_halves_go_to_the_cache(heads, kv, dim, vdim, rot, dty
         q, k = plain.rotate_halves(q, positions, rotation), plain.rotate_halves(k, positions, rotation)
         inv_freq = torch.tensor([77.0 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=F64).float().to(CUDA)
     device = proj.to(dtype).to(CUDA)
-    keys = torch.full((5, kv, page, dim), 9.0, dtype=dtype, device=CUDA)
-    values = torch.full((5, kv, page, vdim), 9.0, dtype=dtype, device=CUDA)
+    keys = torch.full((pages, kv, page, dim), 9.0, dtype=dtype, device=CUDA)
+    values = torch.full((pages, kv, page, vdim), 9.0, dtype=dtype, device=CUDA)
     kernels.qkv_prepare(device, q_at=at, k_at=at + q_cols, v_at=at + q_cols + k_cols, num_q=heads, num_kv=kv, key_dim=dim,
                         value_dim=vdim, positions=ints(positions.tolist()), inv_freq=inv_freq, rot_dims=rot,
                         pairing="half_split", slots=ints(slots), key_cache=keys, value_cache=values, q_bias=qb.to(CUDA),
@@ -479,14 +482,14 @@ def test_biases_and_paired_halves_go_to_the_cache(heads, kv, dim, vdim, rot, dty
     limit = 2e-4 if dtype == torch.float32 else 8e-3             # float32 angles at position 1,000
     close(device[:, at:at + q_cols], q.reshape(tokens, -1), dtype, limit=limit)
     assert torch.equal(device[:, :at].cpu().double(), proj[:, :at])
-    written = torch.zeros(5 * page, dtype=torch.bool)
+    written = torch.zeros(pages * page, dtype=torch.bool)
     for t, slot in enumerate(slots):
         if slot >= 0:
             written[slot] = True
             close(keys[slot // page, :, slot % page], k[t], dtype, limit=limit)
             close(values[slot // page, :, slot % page], v[t], dtype, limit=limit)
-    assert (keys.permute(0, 2, 1, 3).reshape(5 * page, -1)[~written] == 9.0).all()
-    assert (values.permute(0, 2, 1, 3).reshape(5 * page, -1)[~written] == 9.0).all()
+    assert (keys.permute(0, 2, 1, 3).reshape(pages * page, -1)[~written] == 9.0).all()
+    assert (values.permute(0, 2, 1, 3).reshape(pages * page, -1)[~written] == 9.0).all()
 
 
 # ------------------------------------------------------- parts outside the blocks this design puts them in

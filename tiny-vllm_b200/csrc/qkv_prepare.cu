@@ -55,6 +55,7 @@ template <> __device__ __forceinline__ void store_pair<bf16>(bf16* p, float a, f
 // every warp has one head (a q head, a k head or a v head).  Few heads a block keep the chains of
 // dependent loads short: a decode step has only a handful of tokens to spread over the GPU.
 #define PREP_WARPS 4
+#define PREP_WIDE_HALVES 64   // tokens from which paired halves go to the kernel with a block a token
 
 // PAIRS: pairs of a head a lane holds (heads of up to 64 * PAIRS)
 template <typename T, typename W, int PAIRS>
@@ -338,7 +339,7 @@ extern "C" int tvb_qkv_prepare_biased(void* proj, long long token_stride, int q_
     cudaStream_t s = (cudaStream_t)stream;
     const bool wide = dtype == TVB_BF16 && (key_dim == 16 || key_dim == 32 || key_dim == 64 || key_dim == 128 || key_dim == 256) &&
                       value_dim % 8 == 0 && q_at % 8 == 0 && k_at % 8 == 0 && v_at % 8 == 0 && token_stride % 8 == 0 &&
-                      (uintptr_t)proj % 16 == 0 && (!inv_freq || pairing == PREP_PAIR_INTERLEAVED || rot_dims % 16 == 0) &&
+                      (uintptr_t)proj % 16 == 0 && (!inv_freq || pairing == PREP_PAIR_INTERLEAVED || (rot_dims % 16 == 0 && tokens >= PREP_WIDE_HALVES)) &&
                       (!v_first || ((uintptr_t)v_first % 16 == 0 && v_first_stride % 8 == 0)) &&
                       (!slots || ((uintptr_t)key_cache % 16 == 0 && (uintptr_t)value_cache % 16 == 0));
     if (wide) {
