@@ -187,7 +187,7 @@ def test_short_convolution_from_carried_inputs(taps, channels, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
-@pytest.mark.parametrize("channels,n,rank", [(64, 16, 8), (37, 7, 5), (130, 33, 20), (64, 1, 1), (31, 20, 3), (512, 16, 16),
+@pytest.mark.parametrize("channels,n,rank", [(64, 16, 8), (37, 7, 5), (130, 33, 20), (64, 1, 1), (40, 3, 2), (31, 20, 3), (512, 16, 16),
                                              (72, 40, 9), (48, 24, 12), (20, 64, 8), (40, 128, 4), (24, 100, 6), (16, 256, 2)])
 def test_selective_scan_from_a_carried_state(channels, n, rank, dtype):
     """Five entries of one step from carried states, with every number of lanes; then three steps of single tokens in
@@ -224,8 +224,9 @@ def test_selective_scan_from_a_carried_state(channels, n, rank, dtype):
     dx, dz, dbc = dev(x, dtype), dev(z, dtype), dev(bc, dtype)
     common = dict(a=dev(a), d=dev(d), dt_bias=dev(dt_bias))
     limit = 2e-5 if dtype == torch.float32 else None
-    for lanes, tile in [(0, 0)] + [(lanes, tile) for lanes in (2, 4, 8, 16) for tile in (1, 2)
-                                   if lanes * 16 >= n * tile and (tile == 1 or lanes >= 4)]:
+    fewest = 2 if n <= 2 else 4 if n <= 4 else 8 if n <= 128 else 16
+    for lanes, tile in [(0, 0)] + [(lanes, tile) for lanes in sorted({fewest, 16 if n > 8 else fewest}) for tile in (1, 2)
+                                   if tile == 1 or (lanes >= 8 and lanes * 8 >= n)]:
         device_state = dev(state)
         out = torch.full((tokens, channels + 5), 7.0, dtype=dtype, device=CUDA)
         kernels.selective_scan(dx[:, 1:1 + channels], pre=dev(pre), z=dz[:, 3:3 + channels], b=dbc[:, :n], c=dbc[:, n:2 * n],

@@ -20,6 +20,10 @@
 #define SCAN_BLOCK (SCAN_STATE <= 64 ? 32 : 16)      // tokens that wait in shared memory
 #define SCAN_PAD 4
 #define SCAN_FILL 256                                // CTAs from which the GPU counts as full
+// lanes that share a channel: eight (fewer where the state is smaller), sixteen while SMs would idle otherwise or where
+// the state is larger than eight lanes hold
+constexpr int SCAN_FEWEST = SCAN_STATE <= 2 ? 2 : SCAN_STATE <= 4 ? 4 : SCAN_STATE <= 128 ? 8 : 16;
+constexpr int SCAN_MOST = SCAN_STATE > 8 ? 16 : SCAN_FEWEST;
 #define SCAN_LOG2E 1.4426950408889634f
 
 static_assert(SCAN_STATE >= 1 && SCAN_STATE <= 256, "selective_scan: state size");
@@ -289,7 +293,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) selective_scan_kernel(
 
 // x: [tokens, >= channels]; pre float32 [tokens, channels]; z, b, c as x, each with a row stride; a float32
 // [channels, SCAN_STATE]; d, dt_bias float32 [channels]; state float32 [slots, channels, SCAN_STATE]; out
-// [tokens, >= channels].  `lanes` (0: chosen): 2, 4, 8 or 16 lanes a channel; `tile` (0: chosen): one or two channels a
+// [tokens, >= channels].  `lanes` (0: chosen): SCAN_FEWEST or SCAN_MOST lanes a channel; `tile` (0: chosen): one or two channels a
 // thread; a thread holds at most 16 numbers of state.
 extern "C" int tvb_selective_scan(const void* x, long long x_stride, const float* pre, const void* z, long long z_stride,
                                   const void* b, const void* c, long long bc_stride, const float* a, const float* d,
@@ -299,16 +303,10 @@ extern "C" int tvb_selective_scan(const void* x, long long x_stride, const float
     if (rows <= 0) return 0;
     if (channels <= 0 || rows > 65535 || !state || !a || !d || !pre) return TVB_BAD_ARGUMENT;
     auto ctas = [&](int l, int t) { return (long long)rows * ((channels + SCAN_THREADS / l * t - 1) / (SCAN_THREADS / l * t)); };
-    if (lanes == 0) {
-        // eight lanes (fewer where the state is smaller), sixteen while SMs would idle or where the state needs them;
-        // two channels a thread where there are CTAs in plenty
-        for (lanes = 2; lanes < 8 && lanes < SCAN_STATE; lanes *= 2) {}
-        while (lanes < 16 && (lanes * 16 < SCAN_STATE || (lanes < SCAN_STATE && ctas(lanes, 1) < SCAN_FILL))) lanes *= 2;
-    }
-    if (tile == 0) tile = lanes >= 4 && 16 * lanes >= 2 * SCAN_STATE && ctas(lanes, 2) >= 4 * SCAN_FILL ? 2 : 1;
-    if ((lanes != 2 && lanes != 4 && lanes != 8 && lanes != 16) || lanes * 16 < SCAN_STATE * tile || tile < 1 || tile > 2 ||
-        (tile == 2 && lanes < 4))
-        return TVB_BAD_ARGUMENT;
+    if (lanes == 0) lanes = SCAN_MOST > SCAN_FEWEST && ctas(SCAN_FEWEST, 1) < SCAN_FILL ? SCAN_MOST : SCAN_FEWEST;
+    const bool pairs = lanes >= 8 && 16 * lanes >= 2 * SCAN_STATE;        // two channels a thread where CTAs are plenty
+    if (tile == 0) tile = pairs && ctas(lanes, 2) >= 4 * SCAN_FILL ? 2 : 1;
+    if ((lanes != SCAN_FEWEST && lanes != SCAN_MOST) || tile < 1 || tile > 2 || (tile == 2 && !pairs)) return TVB_BAD_ARGUMENT;
     const int ch = SCAN_THREADS / lanes * tile;
     const dim3 grid((channels + ch - 1) / ch, rows);
     cudaStream_t s = (cudaStream_t)stream;
@@ -321,18 +319,13 @@ extern "C" int tvb_selective_scan(const void* x, long long x_stride, const float
         (const T*)x, x_stride, pre, (const T*)z, z_stride, (const T*)b, (const T*)c, bc_stride, a, d, dt_bias, state, \
         row_starts, state_slots, token_row, (T*)out, out_stride, channels)
 #define BY_TILE(T, L)                                                                 \
-    if constexpr (SCAN_STATE * 2 <= 16 * L && L >= 4) {                               \
+    if constexpr (SCAN_STATE * 2 <= 16 * L && L >= 8) {                               \
         if (tile == 2) { GO(T, L, 2); } else { GO(T, L, 1); }                         \
     } else { GO(T, L, 1); }
 #define BY_LANES(T)                                                                   \
-    if (lanes == 16) { BY_TILE(T, 16) }                                               \
-    else if constexpr (SCAN_STATE <= 128) {                                           \
-        if (lanes == 8) { BY_TILE(T, 8) }                                             \
-        else if constexpr (SCAN_STATE <= 64) {                                        \
-            if (lanes == 4) { BY_TILE(T, 4) }                                         \
-            else if constexpr (SCAN_STATE <= 32) { BY_TILE(T, 2) }                    \
-        }                                                                             \
-    }
+    if constexpr (SCAN_MOST > SCAN_FEWEST) {                                          \
+        if (lanes == SCAN_MOST) { BY_TILE(T, SCAN_MOST) } else { BY_TILE(T, SCAN_FEWEST) } \
+    } else { BY_TILE(T, SCAN_FEWEST) }
     if (dtype == TVB_F32) { BY_LANES(float) }
     else if (dtype == TVB_BF16) { BY_LANES(bf16) }
     else return TVB_BAD_ARGUMENT;

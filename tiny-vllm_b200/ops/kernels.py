@@ -1080,8 +1080,9 @@ def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor
     b and c alike), ``pre`` float32 [tokens, channels], ``a`` float32 [channels, n], ``d`` and ``dt_bias`` float32
     [channels].  ``single``: every entry is one token, one launch that reads and writes the state once; instead of
     ``pre`` it may take ``low`` [tokens, rank] (rows apart as those of b) and ``dt_weight`` [channels, rank] and do the
-    product itself.  ``lanes`` (2, 4, 8, 16; 0: chosen): the lanes of a scan that share a
-    channel, ``tile`` (1, 2; 0: chosen): the channels a thread takes."""
+    product itself.  ``lanes`` (0: chosen; 8, or 2 or 4 for states of so few
+    numbers, or 16 for states of more than 8): the lanes of a scan that share a channel, ``tile`` (1, 2; 0: chosen): the
+    channels a thread takes."""
     _need_cuda(x, pre, z, b, c, a, d, dt_bias, state, row_starts, state_slots, token_row, out, low, dt_weight)
     tokens, channels = x.shape
     n = a.shape[1]
