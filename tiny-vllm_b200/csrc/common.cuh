@@ -29,6 +29,24 @@ template <typename T> __device__ __forceinline__ float round_to(float v) {
     return to_float<T>(from_float<T>(v));
 }
 
+// The special-function unit's 2^x and 1 / x: float32, a few units in the last place, tiny results are zero.
+__device__ __forceinline__ float exp2_unit(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float reciprocal_unit(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+// z / (1 + exp(-z)) for a result that is stored as T: with the accurate functions for float32, else with the unit's.
+template <typename T> __device__ __forceinline__ float silu_for(float z);
+template <> __device__ __forceinline__ float silu_for<float>(float z) { return __fdiv_rn(z, __fadd_rn(1.0f, expf(-z))); }
+template <> __device__ __forceinline__ float silu_for<bf16>(float z) {
+    return __fmul_rn(z, reciprocal_unit(1.0f + exp2_unit(__fmul_rn(-z, 1.4426950408889634f))));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int delta = 16; delta > 0; delta >>= 1) v += __shfl_xor_sync(0xffffffffu, v, delta);

@@ -32,34 +32,22 @@ static_assert(SCAN_STATE >= 1 && SCAN_STATE <= 256, "selective_scan: state size"
 // in the last place, far below the rounding of what goes in); decays are then prepared as a log2 e.
 //   decay     exp(dt * a)
 //   softplus  max(z, 0) + ln(1 + exp(-|z|))
-//   silu      z / (1 + exp(-z))
 template <typename T> struct Scan;
 template <> struct Scan<float> {
     static __device__ __forceinline__ float prepare(float a) { return a; }
     static __device__ __forceinline__ float decay(float dt, float a) { return expf(__fmul_rn(dt, a)); }
     static __device__ __forceinline__ float softplus(float z) { return __fadd_rn(fmaxf(z, 0.0f), log1pf(expf(-fabsf(z)))); }
-    static __device__ __forceinline__ float silu(float z) { return __fdiv_rn(z, __fadd_rn(1.0f, expf(-z))); }
 };
 template <> struct Scan<bf16> {
-    static __device__ __forceinline__ float exp2_of(float x) {
-        float y;
-        asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-        return y;
-    }
     static __device__ __forceinline__ float prepare(float a) { return __fmul_rn(a, SCAN_LOG2E); }
-    static __device__ __forceinline__ float decay(float dt, float a) { return exp2_of(__fmul_rn(dt, a)); }
+    static __device__ __forceinline__ float decay(float dt, float a) { return exp2_unit(__fmul_rn(dt, a)); }
     static __device__ __forceinline__ float softplus(float z) {
-        const float u = exp2_of(__fmul_rn(-fabsf(z), SCAN_LOG2E));
+        const float u = exp2_unit(__fmul_rn(-fabsf(z), SCAN_LOG2E));
         float log2;
         asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(log2) : "f"(1.0f + u));
         // the series of ln(1 + u) where 1 + u would round u away
         const float series = u * __fmaf_rn(u, __fmaf_rn(u, __fmaf_rn(u, -0.25f, 0.33333333f), -0.5f), 1.0f);
         return fmaxf(z, 0.0f) + (u < 0.015625f ? series : __fmul_rn(log2, 0.69314718f));
-    }
-    static __device__ __forceinline__ float silu(float z) {
-        float inverse;
-        asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(inverse) : "f"(1.0f + exp2_of(__fmul_rn(-z, SCAN_LOG2E))));
-        return __fmul_rn(z, inverse);
     }
 };
 
@@ -278,7 +266,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) selective_scan_kernel(
                 float y[BOTH];
 #pragma unroll
                 for (int i = 0; i < BOTH; ++i)
-                    y[i] = __fmul_rn(__fmaf_rn(skip[i], x_now[j].at(i), u_s[move_ch + i][t]), Scan<T>::silu(z_now[j].at(i)));
+                    y[i] = __fmul_rn(__fmaf_rn(skip[i], x_now[j].at(i), u_s[move_ch + i][t]), silu_for<T>(z_now[j].at(i)));
                 store_both<BOTH>(dst + j * out_step, y);
             }
         }
@@ -447,7 +435,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) selective_step_kernel(
         if (q < here && live && lane == 0) {
             float result = 0.0f;
             if (owned[q])
-                result = __fmul_rn(__fmaf_rn(skip, xv, y), Scan<T>::silu(to_float<T>(z[(int64_t)token[q] * z_stride + channel])));
+                result = __fmul_rn(__fmaf_rn(skip, xv, y), silu_for<T>(to_float<T>(z[(int64_t)token[q] * z_stride + channel])));
             out[(int64_t)token[q] * out_stride + channel] = from_float<T>(result);
         }
     }

@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
 #pragma unroll
                 for (int j = 0; j < K - 1; ++j) sum = __fmaf_rn(w[j][v], last[j][v], sum);
                 sum = __fmaf_rn(w[K - 1][v], now[t][v], sum);
-                y[v] = act ? __fdiv_rn(sum, __fadd_rn(1.0f, expf(-sum))) : sum;
+                y[v] = act ? silu_for<T>(sum) : sum;
             }
 #pragma unroll
             for (int j = 0; j + 1 < K - 1; ++j)
