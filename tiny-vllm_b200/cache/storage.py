@@ -14,20 +14,34 @@ kv_heads, head_dim]`` (tinyvllm/paged_kv.py:53-65).
 
 from __future__ import annotations
 
+from dataclasses import replace
+
 import torch
 
-from ..parts.base import kv_need, state_needs
+from ..parts.base import KVNeed, kv_need, state_needs
 from .manager import CacheGroup
+
+
+def widened(need: KVNeed, reader: KVNeed) -> KVNeed:
+    """``need`` with a window and first tokens that also hold what ``reader`` sees."""
+    if need.window is None or reader.window is None:
+        return replace(need, window=None, keep_first=0)
+    return replace(need, window=max(need.window, reader.window), keep_first=max(need.keep_first, reader.keep_first))
 
 
 def group_runs(needs: list, cache_from: list) -> tuple[list[CacheGroup], dict[int, tuple[int, int]]]:
     """Groups of equal KV need, and for every run that attends over a cache the
-    (group, index inside the group) of the cache it reads."""
+    (group, index inside the group) of the cache it reads.  A run that reads another's cache may have a window of its
+    own: the cache is kept as long as the widest window over it."""
     groups: list = []
     geometries: list[tuple] = []
     members: list[list[int]] = []
     where: dict[int, tuple[int, int]] = {}
     needs = [kv_need(need) for need in needs]
+    # a cache that later runs read keeps what the widest of all their windows still sees
+    for run, source in enumerate(cache_from):
+        if source is not None and needs[run] is not None and needs[source] is not None:
+            needs[source] = widened(needs[source], needs[run])
     for run, need in enumerate(needs):
         if need is None or cache_from[run] is not None:
             continue
@@ -53,8 +67,8 @@ def group_runs(needs: list, cache_from: list) -> tuple[list[CacheGroup], dict[in
                 need.num_kv_heads, need.head_dim, need.value_size) != (
                     theirs.num_kv_heads, theirs.head_dim, theirs.value_size):
             raise ValueError(f"run {run} cannot read the cache of run {source}: shapes differ")
-        if need.geometry() != theirs.geometry():
-            raise ValueError(f"run {run} and run {source} must agree on the window")
+        if need.value_offset != theirs.value_offset:
+            raise ValueError(f"run {run} and run {source} must agree on where the values are")
         where[run] = where[source]
     return groups, where
 

@@ -435,9 +435,9 @@ extern "C" int tvb_rotate_heads(const void* src, long long src_token_stride, lon
 
 #define HP_COLUMNS 32          // output columns a block takes (grid.z walks the rest)
 
-template <typename T>
+template <typename T, typename O>
 __global__ void head_product_kernel(const T* x, int64_t x_token_stride, int64_t x_head_stride,
-                                    const T* __restrict__ w, T* out, int64_t out_token_stride,
+                                    const T* __restrict__ w, O* out, int64_t out_token_stride,
                                     int64_t out_head_stride, const T* gate, int64_t gate_token_stride, int tokens,
                                     int n, int k) {
     extern __shared__ float x_rows[];                  // [HP_TOKENS][k]
@@ -472,7 +472,7 @@ __global__ void head_product_kernel(const T* x, int64_t x_token_stride, int64_t 
                 const float g = to_float<T>(gate[(int64_t)(first + lane) * gate_token_stride + (int64_t)head * n + j]);
                 o = __fmul_rn(o, __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-g))));
             }
-            out[(int64_t)(first + lane) * out_token_stride + head * out_head_stride + j] = from_float<T>(o);
+            out[(int64_t)(first + lane) * out_token_stride + head * out_head_stride + j] = from_float<O>(o);
         }
     }
 }
@@ -482,7 +482,7 @@ __global__ void head_product_kernel(const T* x, int64_t x_token_stride, int64_t 
 extern "C" int tvb_head_product(const void* x, long long x_token_stride, long long x_head_stride, const void* w,
                                 void* out, long long out_token_stride, long long out_head_stride, const void* gate,
                                 long long gate_token_stride, int tokens, int heads, int n, int k, int dtype,
-                                void* stream) {
+                                int out_dtype, void* stream) {
     if (tokens <= 0) return 0;
     if (heads <= 0 || heads > 65535 || n <= 0 || k <= 0) return TVB_BAD_ARGUMENT;
     const size_t smem = (size_t)HP_TOKENS * k * sizeof(float);
@@ -490,11 +490,12 @@ extern "C" int tvb_head_product(const void* x, long long x_token_stride, long lo
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid((tokens + HP_TOKENS - 1) / HP_TOKENS, heads, (n + HP_COLUMNS - 1) / HP_COLUMNS);
     if (grid.z > 65535) return TVB_BAD_ARGUMENT;
-#define GO(T) head_product_kernel<T><<<grid, HP_WARPS * 32, smem, s>>>(                                          \
-        (const T*)x, x_token_stride, x_head_stride, (const T*)w, (T*)out, out_token_stride, out_head_stride,     \
+#define GO(T, O) head_product_kernel<T, O><<<grid, HP_WARPS * 32, smem, s>>>(                                    \
+        (const T*)x, x_token_stride, x_head_stride, (const T*)w, (O*)out, out_token_stride, out_head_stride,     \
         (const T*)gate, gate_token_stride, tokens, n, k)
-    if (dtype == TVB_F32) GO(float);
-    else if (dtype == TVB_BF16) GO(bf16);
+    if (dtype == TVB_F32 && out_dtype == TVB_F32) GO(float, float);
+    else if (dtype == TVB_BF16 && out_dtype == TVB_BF16) GO(bf16, bf16);
+    else if (dtype == TVB_BF16 && out_dtype == TVB_F32) GO(bf16, float);
     else return TVB_BAD_ARGUMENT;
 #undef GO
     return tvb_last_error();

@@ -36,6 +36,42 @@ extern "C" int tvb_embed_rows(const void* table, const int* ids, void* out, int 
     return tvb_last_error();
 }
 
+// stream[t] = table[ids[t]] * scale in float32, and, where `rounded` is given, its rounding to T.
+template <typename T, int VEC>
+__global__ void embed_scaled_kernel(const T* __restrict__ table, const int* __restrict__ ids, float scale,
+                                    float* __restrict__ stream, T* __restrict__ rounded, int width, int vocab) {
+    const int64_t row = blockIdx.x;
+    int id = ids[row];
+    if (id < 0 || id >= vocab) id = 0;   // the host validates ids; padding rows carry 0
+    const T* src = table + (int64_t)id * width;
+    for (int i = threadIdx.x * VEC; i < width; i += blockDim.x * VEC) {
+        float v[VEC];
+        load_values<VEC>(src + i, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v[j] = __fmul_rn(v[j], scale);
+        store_values<VEC>(stream + row * width + i, v);
+        if (rounded) store_values<VEC>(rounded + row * width + i, v);
+    }
+}
+
+extern "C" int tvb_embed_scaled(const void* table, const int* ids, float scale, float* out, void* rounded, int rows,
+                                int width, int vocab, int dtype, void* stream) {
+    if (rows <= 0) return 0;
+    if (width <= 0 || vocab <= 0 || !out) return TVB_BAD_ARGUMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t element = dtype == TVB_BF16 ? 2 : 4;
+    const bool by_four = width % 4 == 0 && (uintptr_t)table % (4 * element) == 0 && (uintptr_t)rounded % (4 * element) == 0 &&
+                         (uintptr_t)out % 16 == 0;
+    const int per = by_four ? width / 4 : width;
+    const int threads = per >= 512 ? 256 : (per >= 128 ? 128 : 64);
+#define GO(T, VEC) embed_scaled_kernel<T, VEC><<<rows, threads, 0, s>>>((const T*)table, ids, scale, out, (T*)rounded, width, vocab)
+    if (dtype == TVB_F32) { if (by_four) GO(float, 4); else GO(float, 1); }
+    else if (dtype == TVB_BF16) { if (by_four) GO(bf16, 4); else GO(bf16, 1); }
+    else return TVB_BAD_ARGUMENT;
+#undef GO
+    return tvb_last_error();
+}
+
 // out[t] = table[ids[t]] + pairs[(prev * mul_prev + ids[t] * mul_cur) mod buckets] in float32, prev being the
 // token before t in its request: the step's own, or, for the first token of an entry, the one `state`
 // [slots] keeps from the step before.  A request's first token (position 0) reads the last row, number

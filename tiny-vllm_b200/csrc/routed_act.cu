@@ -308,16 +308,21 @@ extern "C" int tvb_route_gated_act(const float* logits, long long logits_stride,
 // scores are chosen (of equal scores the lower index wins).  A chosen slot's weight is s_e as it is, or, with
 // `renormalise`, s_e over the sum of the chosen s.
 //
+// With `groups` > 1 the slots form that many equal groups of neighbours; a group's score is its largest choice
+// score, and only slots of the `keep` best groups can be chosen.
+//
 // The packed projection of a token holds [gate_e | up_e] (ff columns each) expert after expert; column c of
 // expert e of the output holds act(gate) * up times the expert's weight (exactly 0 if the expert was not
-// chosen), act = SiLU.  `identity_out[token]` receives the sum of the chosen pass-through slots' weights: the
+// chosen), act = SiLU; CLIPPED: g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit) and u = clamp(up, -limit,
+// limit) instead.  `identity_out[token]` receives the sum of the chosen pass-through slots' weights: the
 // caller adds that many times the layer's input to the result of the down-projection.
-template <typename T, bool WIDE>
+template <typename T, bool WIDE, bool CLIPPED>
 __global__ void route_softmax_gated_kernel(const float* __restrict__ logits, int64_t logits_stride,
                                            const float* __restrict__ correction, const T* proj, int64_t proj_stride,
                                            T* __restrict__ out, int64_t out_stride, float* __restrict__ weights_out,
                                            float* __restrict__ identity_out, int experts, int identity, int top,
-                                           int renormalise, int ff) {
+                                           int renormalise, int groups, int keep, float limit, float alpha, int ff) {
+    __shared__ float group_score[ROUTE_MAX_EXPERTS];
     __shared__ float share[ROUTE_MAX_EXPERTS];       // softmax scores, then the weight of every slot, 0 if not chosen
     __shared__ float value[ROUTE_MAX_EXPERTS];       // choice scores, -inf once chosen
     __shared__ unsigned char chosen[ROUTE_MAX_EXPERTS];
@@ -344,6 +349,39 @@ __global__ void route_softmax_gated_kernel(const float* __restrict__ logits, int
             value[e] = correction ? __fadd_rn(s, correction[e]) : s;
         }
         __syncwarp();
+        if (groups > 1 && keep < groups) {
+            const int size = slots / groups;
+            for (int g = lane; g < groups; g += 32) {
+                float best = value[g * size];
+                for (int e = g * size + 1; e < (g + 1) * size; ++e) best = fmaxf(best, value[e]);
+                group_score[g] = best;
+            }
+            __syncwarp();
+            // the best groups are marked +inf, one a round (of equal scores the lower index); the others are shut out
+            for (int round = 0; round < keep; ++round) {
+                float best = -INFINITY;
+                int where = ROUTE_MAX_EXPERTS;
+                for (int g = lane; g < groups; g += 32) {
+                    const float c = group_score[g];
+                    if (c != INFINITY && (c > best || where == ROUTE_MAX_EXPERTS)) { best = c; where = g; }
+                }
+#pragma unroll
+                for (int delta = 16; delta > 0; delta >>= 1) {
+                    const float other = __shfl_xor_sync(0xffffffffu, best, delta);
+                    const int other_where = __shfl_xor_sync(0xffffffffu, where, delta);
+                    if (other_where < ROUTE_MAX_EXPERTS &&
+                        (where == ROUTE_MAX_EXPERTS || other > best || (other == best && other_where < where))) {
+                        best = other; where = other_where;
+                    }
+                }
+                if (where >= groups) break;
+                if (lane == 0) group_score[where] = INFINITY;
+                __syncwarp();
+            }
+            for (int e = lane; e < slots; e += 32)
+                if (group_score[e / size] != INFINITY) value[e] = -INFINITY;
+            __syncwarp();
+        }
         float sum = 0.0f;
         for (int round = 0; round < top; ++round) {
             float best = -INFINITY;
@@ -399,8 +437,14 @@ __global__ void route_softmax_gated_kernel(const float* __restrict__ logits, int
                 u[0] = to_float<T>(up[0]);
             }
 #pragma unroll
-            for (int i = 0; i < STEP; ++i)
-                o[i] = __fmul_rn(__fmul_rn(__fdiv_rn(g[i], __fadd_rn(1.0f, expf(-g[i]))), u[i]), weight);
+            for (int i = 0; i < STEP; ++i) {
+                if constexpr (CLIPPED) {
+                    const float gg = fminf(g[i], limit), uu = fminf(fmaxf(u[i], -limit), limit);
+                    const float sig = __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-__fmul_rn(alpha, gg))));
+                    o[i] = __fmul_rn(__fmul_rn(__fmul_rn(gg, sig), __fadd_rn(uu, 1.0f)), weight);
+                } else
+                    o[i] = __fmul_rn(__fmul_rn(__fdiv_rn(g[i], __fadd_rn(1.0f, expf(-g[i]))), u[i]), weight);
+            }
         }
         if constexpr (WIDE) *reinterpret_cast<uint4*>(dst + c) = pack_bf16x8(o);
         else dst[c] = from_float<T>(o[0]);
@@ -409,14 +453,15 @@ __global__ void route_softmax_gated_kernel(const float* __restrict__ logits, int
 
 // logits float32 [tokens, experts + identity]; correction float32 [experts + identity] or null; proj
 // [tokens, 2 * experts * ff] and out [tokens, experts * ff] with row strides; weights_out (optional) float32
-// [tokens, experts + identity]; identity_out (needed with identity > 0) float32 [tokens].
+// [tokens, experts + identity]; identity_out (needed with identity > 0) float32 [tokens]; limit > 0: the clipped form.
 extern "C" int tvb_route_softmax_gated(const float* logits, long long logits_stride, const float* correction,
                                        const void* proj, long long proj_stride, void* out, long long out_stride,
                                        float* weights_out, float* identity_out, int tokens, int experts, int identity,
-                                       int top, int renormalise, int ff, int dtype, void* stream) {
+                                       int top, int renormalise, int groups, int keep, float limit, float alpha, int ff,
+                                       int dtype, void* stream) {
     if (tokens <= 0) return 0;
     if (experts <= 0 || identity < 0 || experts + identity > ROUTE_MAX_EXPERTS || top <= 0 || ff <= 0 ||
-        (identity > 0 && !identity_out))
+        groups <= 0 || (experts + identity) % groups || keep <= 0 || keep > groups || (identity > 0 && !identity_out))
         return TVB_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const long long columns = (long long)experts * ff;
@@ -428,12 +473,14 @@ extern "C" int tvb_route_softmax_gated(const float* logits, long long logits_str
     const dim3 grid(tokens, (unsigned)split);
     const bool wide = dtype == TVB_BF16 && ff % 8 == 0 && proj_stride % 8 == 0 && out_stride % 8 == 0 &&
                       (uintptr_t)proj % 16 == 0 && (uintptr_t)out % 16 == 0;
-#define GO(T, WIDE) route_softmax_gated_kernel<T, WIDE><<<grid, threads, 0, s>>>(                                  \
+#define GO(T, WIDE, CLIPPED) route_softmax_gated_kernel<T, WIDE, CLIPPED><<<grid, threads, 0, s>>>(                \
         logits, logits_stride, correction, (const T*)proj, proj_stride, (T*)out, out_stride, weights_out,          \
-        identity_out, experts, identity, top, renormalise, ff)
-    if (dtype == TVB_F32) GO(float, false);
-    else if (dtype == TVB_BF16) { if (wide) GO(bf16, true); else GO(bf16, false); }
+        identity_out, experts, identity, top, renormalise, groups, keep, limit, alpha, ff)
+#define BY_FORM(T, WIDE) if (limit > 0.0f) GO(T, WIDE, true); else GO(T, WIDE, false)
+    if (dtype == TVB_F32) { BY_FORM(float, false); }
+    else if (dtype == TVB_BF16) { if (wide) { BY_FORM(bf16, true); } else { BY_FORM(bf16, false); } }
     else return TVB_BAD_ARGUMENT;
+#undef BY_FORM
 #undef GO
     return tvb_last_error();
 }

@@ -2,6 +2,8 @@
 //
 //   y[t, c] = act(bias[c] + sum_j taps[j, c] * x[t - (K - 1) + j, c])        act none or SiLU
 //
+// With `in_bias` the inputs are x + in_bias (the zeros before a request's start stay zeros).
+//
 // The inputs before a step's first token are the request's last K - 1 ones, kept in a float32 state
 // [slots, K - 1, channels] (oldest first, zero when a request starts), which is left as the last K - 1
 // inputs of the entry.  K is 2, 4, 8, 16 or 32; fewer taps are padded with zeros in front (the older ones).
@@ -18,8 +20,8 @@ template <int K> constexpr int CONV_PIECE = K <= 8 ? 8 : 32;
 
 template <typename T, int K, int VEC>
 __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
-    const T* __restrict__ x, int64_t x_stride, const float* __restrict__ taps, const float* __restrict__ bias, int act,
-    float* state, const int* __restrict__ row_starts, const int* __restrict__ state_slots,
+    const T* __restrict__ x, int64_t x_stride, const float* __restrict__ taps, const float* __restrict__ bias,
+    const float* __restrict__ in_bias, int act, float* state, const int* __restrict__ row_starts, const int* __restrict__ state_slots,
     const int* __restrict__ token_row, T* __restrict__ out, int64_t out_stride, int rows, int channels) {
     const int c = (blockIdx.x * CONV_THREADS + threadIdx.x) * VEC;
     constexpr int PIECE = CONV_PIECE<K>;
@@ -42,15 +44,23 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
     }
     const T* src = x + (int64_t)begin * x_stride + c;
     float* mine = state + (int64_t)state_slots[row] * (K - 1) * channels + c;
-    float w[K][VEC], b[VEC] = {}, last[K - 1][VEC];
+    float w[K][VEC], b[VEC] = {}, shift[VEC] = {}, last[K - 1][VEC];
+    auto input = [&](const T* p, float* v) {
+        load_values<VEC>(p, v);
+        if (in_bias) {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] = __fadd_rn(v[i], shift[i]);
+        }
+    };
 #pragma unroll
     for (int j = 0; j < K; ++j) load_values<VEC>(taps + (int64_t)j * channels + c, w[j]);
     if (bias) load_values<VEC>(bias + c, b);
+    if (in_bias) load_values<VEC>(in_bias + c, shift);
 #pragma unroll
     for (int j = 0; j < K - 1; ++j) {
         const int i = i0 - (K - 1) + j;           // before the entry's first token only in its first piece
         if (i < 0) load_values<VEC>(mine + (int64_t)(K - 1 + i) * channels, last[j]);
-        else load_values<VEC>(src + (int64_t)i * x_stride, last[j]);
+        else input(src + (int64_t)i * x_stride, last[j]);
     }
     if (piece == 0) {
 #pragma unroll
@@ -58,7 +68,7 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
             const int i = tokens - (K - 1) + j;
             float v[VEC];
             if (i < 0) load_values<VEC>(mine + (int64_t)(K - 1 + i) * channels, v);
-            else load_values<VEC>(src + (int64_t)i * x_stride, v);
+            else input(src + (int64_t)i * x_stride, v);
             store_values<VEC>(mine + (int64_t)j * channels, v);
         }
     }
@@ -67,7 +77,7 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
         float now[8][VEC];
 #pragma unroll
         for (int t = 0; t < 8; ++t)
-            if (t0 + t < count) load_values<VEC>(src + (int64_t)(t0 + t) * x_stride, now[t]);
+            if (t0 + t < count) input(src + (int64_t)(t0 + t) * x_stride, now[t]);
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
             if (t0 + t >= count) break;
@@ -92,9 +102,9 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(
 }
 
 // x: the first channel of the first token, rows `x_stride` elements apart; taps float32 [taps_count, channels];
-// bias float32 [channels] or null; act 0 none, 1 SiLU; `tokens`: of all entries.
+// bias and in_bias float32 [channels] or null; act 0 none, 1 SiLU; `tokens`: of all entries.
 extern "C" int tvb_short_conv(const void* x, long long x_stride, const float* taps, int taps_count, const float* bias,
-                              int act, float* state, const int* row_starts, const int* state_slots,
+                              const float* in_bias, int act, float* state, const int* row_starts, const int* state_slots,
                               const int* token_row, void* out, long long out_stride, int rows, int tokens, int channels,
                               int dtype, void* stream) {
     if (rows <= 0 || tokens <= 0) return 0;
@@ -102,14 +112,15 @@ extern "C" int tvb_short_conv(const void* x, long long x_stride, const float* ta
     const size_t element = dtype == TVB_BF16 ? 2 : 4;
     const bool by_four = taps_count <= 8 && channels % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 &&
                          (uintptr_t)x % (4 * element) == 0 && (uintptr_t)out % (4 * element) == 0 &&
-                         (uintptr_t)taps % 16 == 0 && (uintptr_t)bias % 16 == 0 && (uintptr_t)state % 16 == 0;
+                         (uintptr_t)taps % 16 == 0 && (uintptr_t)bias % 16 == 0 && (uintptr_t)in_bias % 16 == 0 &&
+                         (uintptr_t)state % 16 == 0;
     const int per = CONV_THREADS * (by_four ? 4 : 1);
     const long long pieces = tokens / (taps_count <= 8 ? 8 : 32) + (long long)rows;        // at least those of all entries
     if (pieces > 65535) return TVB_BAD_ARGUMENT;
     const dim3 grid((channels + per - 1) / per, (unsigned)pieces);
     cudaStream_t s = (cudaStream_t)stream;
 #define GO(T, K, VEC) short_conv_kernel<T, K, VEC><<<grid, CONV_THREADS, 0, s>>>(                                     \
-        (const T*)x, x_stride, taps, bias, act, state, row_starts, state_slots, token_row, (T*)out, out_stride, rows, channels)
+        (const T*)x, x_stride, taps, bias, in_bias, act, state, row_starts, state_slots, token_row, (T*)out, out_stride, rows, channels)
 #define BY_TAPS(T)                                                                                                     \
     switch (taps_count) {                                                                                              \
         case 2: if (by_four) GO(T, 2, 4); else GO(T, 2, 1); break;                                                     \

@@ -84,7 +84,7 @@ extern "C" int tvb_stream_norm(const float* stream_in, const void* add1, const v
 // ---------------------------------------------- a norm after a sublayer and the norm before the next
 //   sandwich_norm   t  = y + scale[row] * x                    (the second term optional)
 //                   s' = s + t * rsqrt(mean(t^2) + eps_post) * w_post     (without w_post: s' = s + t; without y: s' = s)
-//                   out = round_T(s' * rsqrt(mean(s'^2) + eps_pre) * w_pre)   (without w_pre: no out)
+//                   out = round_T(s' * rsqrt(mean(s'^2) + eps_pre) * w_pre)   (without w_pre: round_T(s'), or no out)
 //                   One block per row, all of it float32 with one rounding at the end.  A sublayer's output
 //                   is normed before it joins the stream, and the stream is normed for the next sublayer, in
 //                   one pass over the row.  With `gather` only the named rows are produced and the stream is
@@ -179,10 +179,10 @@ __global__ void sandwich_norm_kernel(const float* stream_in, const Y* y, const f
             if constexpr (VEC == 4) store4(stream_out + (int64_t)out_row * width + i, v);
             else stream_out[(int64_t)out_row * width + i] = v[0];
         }
-        if (pre_weight) {
-            get(pre_weight + i, w);
+        if (out) {
+            if (pre_weight) get(pre_weight + i, w);
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) o[j] = __fmul_rn(__fmul_rn(v[j], inverse_pre), w[j]);
+            for (int j = 0; j < VEC; ++j) o[j] = pre_weight ? __fmul_rn(__fmul_rn(v[j], inverse_pre), w[j]) : v[j];
             if constexpr (VEC == 4) store4(out + (int64_t)out_row * width + i, o);
             else out[(int64_t)out_row * width + i] = from_float<T>(o[0]);
         }

@@ -278,6 +278,8 @@ def windowed_attention(ctx, mixer, projected: torch.Tensor, at: int, run: int, o
     q_bias, k_bias = getattr(mixer, "q_bias", None), getattr(mixer, "k_bias", None)
     v_bias = getattr(mixer, "v_bias", None)
     bias_table, segment = getattr(mixer, "bias_table", None), getattr(mixer, "segment", None)
+    if writes and getattr(mixer, "reads_other_cache", False):
+        raise kernels.KernelError("a mixer without keys and values runs on another run's cache (cache_from)")
     if values_are_keys and not writes:
         raise kernels.KernelError("values that are the keys need the step's keys written to the cache")
     if mixer.qk_norm == "whole" and (q_bias is not None or values_are_keys):
@@ -313,16 +315,20 @@ def windowed_attention(ctx, mixer, projected: torch.Tensor, at: int, run: int, o
         head_norm = None
         prepared = plain_rest           # nothing is left to rotate or blend: the norm kernel stored k and v itself
     if not prepared:
+        # without a cache write there are no keys to prepare: the run reads those of an earlier one
         kernels.qkv_prepare(
-            projected, q_at=q_at, k_at=k_at, v_at=v_at, num_q=mixer.num_heads, num_kv=mixer.num_kv_heads,
+            projected, q_at=q_at, k_at=k_at, v_at=v_at, num_q=mixer.num_heads,
+            num_kv=mixer.num_kv_heads if writes else 0,
             key_dim=mixer.key_dim, value_dim=mixer.value_dim, positions=ctx.positions, norm=head_norm,
-            q_weight=mixer.q_norm_weight, k_weight=mixer.k_norm_weight, eps=mixer.qk_norm_eps,
+            q_weight=mixer.q_norm_weight, k_weight=mixer.k_norm_weight if writes else mixer.q_norm_weight,
+            eps=mixer.qk_norm_eps,
             inv_freq=None if position is None else position.inv_freq,
             rot_dims=0 if position is None else position.rot_dims,
             pairing="interleaved" if position is None else position.pairing,
             slots=ctx.slots[group] if writes else None, key_cache=keys, value_cache=values,
-            v_first=v_first, blend=mixer.vmix if v_first is not None else None,
-            q_bias=q_bias, k_bias=k_bias, v_bias=k_bias if values_are_keys else v_bias)
+            v_first=v_first if writes else None, blend=mixer.vmix if v_first is not None and writes else None,
+            q_bias=q_bias, k_bias=k_bias if writes else None,
+            v_bias=None if not writes else k_bias if values_are_keys else v_bias)
     gate = projected[:, g_at:g_at + mixer.gate_cols] if mixer.gate else None
     queries = projected[:, q_at:q_at + mixer.q_cols]
     heads = dict(num_q=mixer.num_heads, num_kv=mixer.num_kv_heads, key_dim=mixer.key_dim,

@@ -135,6 +135,22 @@ def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor | None 
 
 
 # -------------------------------------------------------------------- RMSNorm
+def embed_scaled(table: torch.Tensor, ids: torch.Tensor, scale: float):
+    """(stream, rounded): table[ids[t]] * scale in float32, and its rounding to the table's dtype (float32: the
+    stream itself); ids int32."""
+    _need_cuda(table, ids)
+    if ids.dtype != torch.int32 or ids.dim() != 1 or table.dim() != 2 or not table.is_contiguous():
+        raise KernelError("embed_scaled wants a contiguous [vocab, width] table and int32 ids [tokens]")
+    rows, (vocab, width) = ids.shape[0], table.shape
+    out = torch.empty((rows, width), dtype=torch.float32, device=table.device)
+    rounded = None if table.dtype == torch.float32 else torch.empty((rows, width), dtype=table.dtype, device=table.device)
+    fn = _fn("pointwise", "tvb_embed_scaled",
+             [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(table.data_ptr(), ids.data_ptr(), scale, out.data_ptr(), _ptr(rounded), rows, width, vocab,
+              dtype_tag(table.dtype), _stream()), "embed_scaled")
+    return out, (out if rounded is None else rounded)
+
+
 def embed_pairs(table: torch.Tensor, ids: torch.Tensor, *, positions: torch.Tensor, token_row: torch.Tensor,
                 row_starts: torch.Tensor, state_slots: torch.Tensor, pairs: dict | None = None) -> torch.Tensor:
     """float32 [tokens, width]: table[ids[t]], plus, with ``pairs`` (``table`` [buckets + 1, width], ``mul_prev``,
@@ -466,13 +482,14 @@ def stream_norm(stream: torch.Tensor | None, weight: torch.Tensor | None, eps: f
 def sandwich_norm(stream: torch.Tensor, y: torch.Tensor | None, *, post_weight: torch.Tensor | None = None,
                   pre_weight: torch.Tensor | None = None, post_eps: float = 0.0, pre_eps: float = 0.0,
                   row_scale: torch.Tensor | None = None, x: torch.Tensor | None = None,
-                  rows: torch.Tensor | None = None, out_dtype: torch.dtype | None = None):
+                  rows: torch.Tensor | None = None, out_dtype: torch.dtype | None = None, rounded: bool = False):
     """A norm behind a sublayer and the norm in front of the next, in one pass over a float32 residual stream.
 
     t = y + row_scale[:, None] * x (the second term with ``row_scale`` float32 [tokens] and ``x`` [tokens, width]
     of the storage type); s' = stream + t * rsqrt(mean(t^2) + post_eps) * post_weight, written back into
     ``stream`` (without ``post_weight``: s' = stream + t; without ``y``: s' = stream); out = s' * rsqrt(mean(s'^2)
-    + pre_eps) * pre_weight, rounded once to ``out_dtype`` (without ``pre_weight`` no out).  All float32.
+    + pre_eps) * pre_weight, rounded once to ``out_dtype`` (without ``pre_weight``: s' rounded to it with ``rounded``,
+    else no out).  All float32.
     Returns (out, stream).  With ``rows`` (int32) only those rows of out are produced and nothing is written
     back: (out, None)."""
     _need_cuda(stream, y, post_weight, pre_weight, row_scale, x, rows)
@@ -481,6 +498,8 @@ def sandwich_norm(stream: torch.Tensor, y: torch.Tensor | None, *, post_weight: 
     tokens, width = stream.shape
     if y is not None and (y.shape != (tokens, width) or not y.is_contiguous()):
         raise KernelError("sandwich_norm: y must match the stream")
+    if rounded and pre_weight is not None:
+        raise KernelError("sandwich_norm: the result is the normed stream or the rounded one")
     if post_weight is not None and y is None:
         raise KernelError("sandwich_norm: a norm behind the sublayer needs the sublayer's output")
     weights = [w for w in (post_weight, pre_weight) if w is not None]
@@ -498,7 +517,9 @@ def sandwich_norm(stream: torch.Tensor, y: torch.Tensor | None, *, post_weight: 
     if rows is not None and rows.dtype != torch.int32:
         raise KernelError("sandwich_norm: rows must be int32")
     count = tokens if rows is None else rows.shape[0]
-    out = torch.empty((count, width), dtype=out_dtype, device=stream.device) if pre_weight is not None else None
+    out = None
+    if pre_weight is not None or rounded:
+        out = torch.empty((count, width), dtype=out_dtype, device=stream.device)
     fn = _fn("stream_norm", "tvb_sandwich_norm",
              [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p,
               c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p])
@@ -750,7 +771,8 @@ HEAD_PRODUCT_LIBRARY_TOKENS = 64   # bfloat16 tokens from which the products go 
 def head_product(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, gate: torch.Tensor | None = None) -> None:
     """out[t, h, j] = sum_k x[t, h, k] * w[h, j, k] for x [tokens, heads, k] and out [tokens, heads, n] with
     strides of their own and contiguous w [heads, n, k]; with ``gate`` [tokens, heads * n] the result is
-    multiplied by sigmoid(gate) before it is rounded.  float32 sums in an order that k alone fixes."""
+    multiplied by sigmoid(gate) before it is rounded.  float32 sums in an order that k alone fixes.  ``out`` may be
+    float32 beside 16-bit operands (without a gate)."""
     _need_cuda(x, w, out, gate)
     if w.dim() != 3 or not w.is_contiguous():
         raise KernelError("head_product wants contiguous weights [heads, n, k]")
@@ -758,11 +780,12 @@ def head_product(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, gate: t
     tokens = x.shape[0]
     x_strides = _heads_view(x, heads, k, "head_product: x")
     o_strides = _heads_view(out, heads, n, "head_product: out")
-    if out.shape[0] != tokens or not (x.dtype == w.dtype == out.dtype) or k > HEAD_PRODUCT_MAX_K:
+    unrounded = out.dtype == torch.float32 and x.dtype == torch.bfloat16 and gate is None
+    if out.shape[0] != tokens or x.dtype != w.dtype or not (out.dtype == x.dtype or unrounded) or k > HEAD_PRODUCT_MAX_K:
         raise KernelError(f"head_product: one dtype, equal token counts, k up to {HEAD_PRODUCT_MAX_K}")
     if gate is not None and (gate.shape != (tokens, heads * n) or gate.stride(1) != 1 or gate.dtype != x.dtype):
         raise KernelError("head_product: gate must be [tokens, heads * n] of the same dtype with contiguous rows")
-    if x.dtype == torch.bfloat16 and tokens >= HEAD_PRODUCT_LIBRARY_TOKENS:
+    if x.dtype == torch.bfloat16 and tokens >= HEAD_PRODUCT_LIBRARY_TOKENS and not unrounded:
         # many tokens: one batched library product (a batch a head) on the tensor cores, then the result goes
         # to its place, with the gate on the way
         by_head = torch.bmm(x.transpose(0, 1), w.transpose(1, 2))            # [heads, tokens, n]
@@ -774,9 +797,10 @@ def head_product(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, gate: t
         return
     fn = _fn("latent_prepare", "tvb_head_product",
              [c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong,
-              c_int, c_int, c_int, c_int, c_int, c_void_p])
+              c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(x.data_ptr(), *x_strides, w.data_ptr(), out.data_ptr(), *o_strides, _ptr(gate),
-              0 if gate is None else gate.stride(0), tokens, heads, n, k, dtype_tag(x.dtype), _stream()),
+              0 if gate is None else gate.stride(0), tokens, heads, n, k, dtype_tag(x.dtype), dtype_tag(out.dtype),
+              _stream()),
            "head_product")
 
 
@@ -863,16 +887,18 @@ def route_gated_act(logits: torch.Tensor, proj: torch.Tensor, *, experts: int, t
 
 
 def route_softmax_gated(logits: torch.Tensor, proj: torch.Tensor, *, experts: int, identity: int, top: int, ff: int,
-                        correction: torch.Tensor | None = None, renormalise: bool = False,
-                        out: torch.Tensor | None = None, weights_out: torch.Tensor | None = None):
+                        correction: torch.Tensor | None = None, renormalise: bool = False, groups: int = 1, keep: int = 1,
+                        limit: float | None = None, alpha: float = 1.0, out: torch.Tensor | None = None, weights_out: torch.Tensor | None = None):
     """Softmax routing over experts and pass-through slots, and gated experts, between the packed input and
     output products.
 
     ``logits`` float32 [tokens, experts + identity]; the scores are their softmax over all slots, the ``top``
     slots with the largest score + ``correction`` (float32 [experts + identity]) are chosen, and a chosen
-    slot's weight is its score (``renormalise``: over the sum of the chosen scores).  ``proj`` [tokens, 2 *
-    experts * ff] holds [gate | up] of every expert; the result [tokens, experts * ff] holds silu(gate) * up
-    times the expert's weight (0 if not chosen).  The last ``identity`` slots have no columns: the sum of their
+    slot's weight is its score (``renormalise``: over the sum of the chosen scores).  With ``groups`` > 1 only slots
+    of the ``keep`` best of so many equal groups of neighbours can be chosen (a group's score: its largest choice
+    score).  ``proj`` [tokens, 2 * experts * ff] holds [gate | up] of every expert; the result [tokens, experts * ff]
+    holds silu(gate) * up times the expert's weight (0 if not chosen), or, with ``limit``, g * sigmoid(alpha * g) *
+    (u + 1) times it, g = min(gate, limit) and u = clamp(up, -limit, limit).  The last ``identity`` slots have no columns: the sum of their
     weights comes back as float32 [tokens] (None without such slots), and the caller adds that many times the
     experts' input to the down-projection's result.  Returns (inner, identity weights)."""
     _need_cuda(logits, proj, correction, out, weights_out)
@@ -884,6 +910,8 @@ def route_softmax_gated(logits: torch.Tensor, proj: torch.Tensor, *, experts: in
     if proj.dim() != 2 or proj.shape[1] != 2 * columns or proj.stride(1) != 1 or experts <= 0 or identity < 0 \
             or slots > ROUTE_MAX_EXPERTS or top <= 0:
         raise KernelError("route_softmax_gated: the projection must be [tokens, 2 * experts * ff]")
+    if groups <= 0 or slots % groups or not 0 < keep <= groups or (limit is not None and not limit > 0):
+        raise KernelError("route_softmax_gated: slots form equal groups of which some are kept; a limit is positive")
     if correction is not None and (correction.dtype != torch.float32 or correction.shape != (slots,)
                                    or not correction.is_contiguous()):
         raise KernelError("route_softmax_gated: the correction is contiguous float32 [experts + identity]")
@@ -897,10 +925,10 @@ def route_softmax_gated(logits: torch.Tensor, proj: torch.Tensor, *, experts: in
     passed = torch.empty((tokens,), dtype=torch.float32, device=proj.device) if identity else None
     fn = _fn("routed_act", "tvb_route_softmax_gated",
              [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_int,
-              c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+              c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p])
     _check(fn(logits.data_ptr(), logits.stride(0), _ptr(correction), proj.data_ptr(), proj.stride(0),
               out.data_ptr(), out.stride(0), _ptr(weights_out), _ptr(passed), tokens, experts, identity, top,
-              1 if renormalise else 0, ff, dtype_tag(proj.dtype), _stream()), "route_softmax_gated")
+              1 if renormalise else 0, groups, keep, 0.0 if limit is None else limit, alpha, ff, dtype_tag(proj.dtype), _stream()), "route_softmax_gated")
     return out, passed
 
 
@@ -1029,19 +1057,22 @@ def _entry_checks(who: str, tokens: int, row_starts, state_slots, token_row) -> 
 
 def short_convolution(x: torch.Tensor, taps: torch.Tensor, *, bias: torch.Tensor | None, act: str | None,
                       state: torch.Tensor, row_starts: torch.Tensor, state_slots: torch.Tensor,
-                      token_row: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+                      token_row: torch.Tensor, out: torch.Tensor | None = None,
+                      in_bias: torch.Tensor | None = None) -> torch.Tensor:
     """act(bias + sum_j taps[j] * x[t - (K - 1) + j]) per channel: x [tokens, channels] (rows may be strided), taps
     float32 [K, channels] with K one of CONV_TAPS (the last tap is the current token's).  The inputs before an
     entry's first token are those ``state`` (float32 [slots, K - 1, channels], oldest first) keeps in the entry's
-    slot, which is left as the entry's last K - 1 inputs."""
-    _need_cuda(x, taps, bias, state, row_starts, state_slots, token_row, out)
+    slot, which is left as the entry's last K - 1 inputs.  With ``in_bias`` (float32 [channels]) the inputs are x +
+    in_bias (a fresh request's zeros stay zeros)."""
+    _need_cuda(x, taps, bias, state, row_starts, state_slots, token_row, out, in_bias)
     tokens, channels = x.shape
     rows = _entry_checks("short_convolution", tokens, row_starts, state_slots, token_row)
     if x.stride(1) != 1 or taps.dim() != 2 or taps.shape[0] not in CONV_TAPS or taps.shape[1] != channels \
             or taps.dtype != torch.float32 or not taps.is_contiguous():
         raise KernelError(f"short_convolution wants x with contiguous rows and float32 taps [{CONV_TAPS}, channels]")
-    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (channels,) or not bias.is_contiguous()):
-        raise KernelError("short_convolution: the bias is contiguous float32 [channels]")
+    for b in (bias, in_bias):
+        if b is not None and (b.dtype != torch.float32 or b.shape != (channels,) or not b.is_contiguous()):
+            raise KernelError("short_convolution: biases are contiguous float32 [channels]")
     if state.dtype != torch.float32 or state.dim() != 3 or state.shape[1:] != (taps.shape[0] - 1, channels) \
             or not state.is_contiguous():
         raise KernelError("short_convolution: the state is contiguous float32 [slots, K - 1, channels]")
@@ -1052,9 +1083,9 @@ def short_convolution(x: torch.Tensor, taps: torch.Tensor, *, bias: torch.Tensor
     elif out.shape != x.shape or out.dtype != x.dtype or out.stride(1) != 1:
         raise KernelError("short_convolution: out must be [tokens, channels] of the dtype of x")
     fn = _fn("short_conv", "tvb_short_conv",
-             [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-              c_longlong, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(x.data_ptr(), x.stride(0), taps.data_ptr(), taps.shape[0], _ptr(bias), CONV_ACTS[act], state.data_ptr(),
+             [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+              c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(x.data_ptr(), x.stride(0), taps.data_ptr(), taps.shape[0], _ptr(bias), _ptr(in_bias), CONV_ACTS[act], state.data_ptr(),
               row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows,
               tokens, channels, dtype_tag(x.dtype), _stream()), "short_convolution")
     return out
@@ -1132,6 +1163,191 @@ def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor
               b.stride(0), a.data_ptr(), d.data_ptr(), _ptr(dt_bias), state.data_ptr(), row_starts.data_ptr(),
               state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows, channels, lanes, tile, tag,
               _stream()), "selective_scan")
+    return out
+
+
+# ------------------------------------- linear recurrent unit: a number of state a channel, gates from square matrices
+UNIT_ACTS = {None: 0, "silu": 1, "gelu_tanh": 2}
+UNIT_STEP_ROWS = 16               # requests up to which the step kernel does the gates' products itself
+UNIT_STEP_FLOATS = 40 * 1024 // 4  # float32 numbers of u that wait in its shared memory
+
+
+def recurrent_unit_step_takes(rows: int, size: int) -> bool:
+    """Whether a step of single tokens does the gates' products (square matrices of ``size``) inside the step kernel:
+    its CTAs read the weights once for up to eight requests."""
+    together = 1 if rows <= 1 else 2 if rows == 2 else 4 if rows <= 4 else 8
+    return rows <= UNIT_STEP_ROWS and together * (-(-size // 8) * 8) <= UNIT_STEP_FLOATS
+
+
+def block_products(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """float32 [tokens, blocks, n] (any strides): the parts of x [tokens, blocks * size] times w [blocks, n, size]
+    transposed, part by part.  16-bit operands of vector sizes go to one batched library product, everything else to
+    the float32-core kernels."""
+    _need_cuda(x, w)
+    blocks, n, size = w.shape
+    tokens = x.shape[0]
+    if x.dim() != 2 or x.shape[1] != blocks * size or x.stride(1) != 1 or x.dtype != w.dtype or not w.is_contiguous():
+        raise KernelError("block_products wants x [tokens, blocks * size] and contiguous w [blocks, n, size] of one dtype")
+    parts = x.unflatten(1, (blocks, size))
+    if x.dtype == torch.bfloat16 and size % 8 == 0 and n % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0:
+        return torch.bmm(parts.transpose(0, 1), w.transpose(1, 2), out_dtype=torch.float32).transpose(0, 1)
+    out = torch.empty((tokens, blocks, n), dtype=torch.float32, device=x.device)
+    if size <= HEAD_PRODUCT_MAX_K:
+        head_product(parts, w, out)
+    else:
+        for block in range(blocks):
+            gemm_nt_simt(parts[:, block], w[block], out=out[:, block])
+    return out
+
+
+def recurrent_unit(u: torch.Tensor, y: torch.Tensor, *, blocks: int, decay: torch.Tensor, bias_r: torch.Tensor,
+                   bias_i: torch.Tensor, state: torch.Tensor, row_starts: torch.Tensor, state_slots: torch.Tensor,
+                   token_row: torch.Tensor, pre: torch.Tensor | None = None, weight: torch.Tensor | None = None,
+                   bias_y: torch.Tensor | None = None, act: str | None = "gelu_tanh", single: bool = False,
+                   out: torch.Tensor | None = None) -> torch.Tensor:
+    """The linear recurrent unit behind its convolution: r = sigmoid(pre_r + bias_r), i = sigmoid(pre_i + bias_i), a =
+    exp(decay r), S <- a S + sqrt(1 - a^2) i u, out = S act(y + bias_y), a channel by itself, token by token from the
+    float32 ``state`` [slots, channels] of the entry's slot, which is left as the state after the entry's last token.
+
+    ``u``, ``y``, ``out`` [tokens, channels] of the storage type (rows may be strided); ``decay`` (not positive) and the
+    biases float32 [channels].  ``pre`` float32 [tokens, blocks, 2 * size] (any strides; size = channels / blocks): r's
+    pre-activations of every block, then i's.  ``single``: every entry is one token; instead of ``pre`` it may take
+    ``weight`` [blocks, 2 * size, size], whose products with u it does itself."""
+    _need_cuda(u, y, pre, weight, decay, bias_r, bias_i, bias_y, state, row_starts, state_slots, token_row, out)
+    tokens, channels = u.shape
+    rows = _entry_checks("recurrent_unit", tokens, row_starts, state_slots, token_row)
+    if blocks <= 0 or channels % blocks:
+        raise KernelError("recurrent_unit: the channels form equal blocks")
+    size = channels // blocks
+    if out is None:
+        out = torch.empty((tokens, channels), dtype=u.dtype, device=u.device)
+    for name, t in (("u", u), ("y", y), ("out", out)):
+        if t.shape != (tokens, channels) or t.dtype != u.dtype or t.stride(1) != 1:
+            raise KernelError(f"recurrent_unit: {name} must be [tokens, channels] of one dtype with contiguous rows")
+    for name, t in (("decay", decay), ("bias_r", bias_r), ("bias_i", bias_i), ("bias_y", bias_y)):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (channels,) or not t.is_contiguous()):
+            raise KernelError(f"recurrent_unit: {name} must be contiguous float32 [channels]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] != channels or not state.is_contiguous():
+        raise KernelError("recurrent_unit: the state is contiguous float32 [slots, channels]")
+    if act not in UNIT_ACTS:
+        raise KernelError(f"recurrent_unit: the activation {act!r} is not known")
+    if (pre is None) == (weight is None) or (weight is not None and not single):
+        raise KernelError("recurrent_unit takes either pre or, for single tokens, weight")
+    if single and tokens != rows:
+        raise KernelError("recurrent_unit: a step of single tokens has as many tokens as entries")
+    if pre is not None and (pre.dtype != torch.float32 or pre.shape != (tokens, blocks, 2 * size) or pre.stride(2) != 1):
+        raise KernelError("recurrent_unit: pre must be float32 [tokens, blocks, 2 * size]")
+    if weight is not None and (weight.dtype != u.dtype or weight.shape != (blocks, 2 * size, size)
+                               or not weight.is_contiguous() or not recurrent_unit_step_takes(min(rows, UNIT_STEP_ROWS), size)):
+        raise KernelError("recurrent_unit: weight must be contiguous [blocks, 2 * size, size] of the dtype of u, of a "
+                          "size that waits in shared memory")
+    fn = _fn("recurrent_unit", "tvb_recurrent_unit",
+             [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p,
+              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
+              c_int, c_int, c_void_p])
+    _check(fn(u.data_ptr(), u.stride(0), y.data_ptr(), y.stride(0), _ptr(pre), 0 if pre is None else pre.stride(0),
+              0 if pre is None else pre.stride(1), _ptr(weight), bias_r.data_ptr(), bias_i.data_ptr(), decay.data_ptr(),
+              _ptr(bias_y), state.data_ptr(), row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(),
+              out.data_ptr(), out.stride(0), rows, channels, size, UNIT_ACTS[act], 1 if single else 0, dtype_tag(u.dtype),
+              _stream()), "recurrent_unit")
+    return out
+
+
+# ------------------------------------------------------------------------------------- gated delta rule
+DELTA_MAX_DIM = 256
+DELTA_MAX_STEP_GROUPS = 256       # columns (in fours, where they fit) of a head that the step kernel takes
+
+
+def delta_step_takes(dim: int, vdim: int) -> bool:
+    """Whether a step of single tokens of :func:`delta_rule` runs as one launch."""
+    groups = vdim // 4 if vdim % 4 == 0 else vdim
+    slices = max(1, DELTA_MAX_STEP_GROUPS // max(groups, 1))
+    floats = 2 * dim + 2 * vdim + 2 * slices * vdim
+    return groups <= DELTA_MAX_STEP_GROUPS and floats * 4 <= 48 * 1024
+
+
+def delta_rule(mixed: torch.Tensor, proj: torch.Tensor, *, q_at: int, k_at: int, v_at: int, beta_at: int, decay_at: int,
+               heads: int, key_heads: int, dim: int, vdim: int, rate: torch.Tensor, dt_bias: torch.Tensor,
+               state: torch.Tensor, row_starts: torch.Tensor, state_slots: torch.Tensor, token_row: torch.Tensor,
+               query_scale: float = 1.0, unit_eps: float = 1e-6, unit_norm: bool = True,
+               norm_weight: torch.Tensor | None = None, eps: float = 0.0, gate_at: int | None = None,
+               gate_act: str | None = "silu", out: torch.Tensor | None = None,
+               raw_out: torch.Tensor | None = None) -> torch.Tensor:
+    """The gated delta rule between a mixer's convolution and its output projection.
+
+    ``mixed`` [tokens, columns] (convolved) holds q heads (``key_heads`` of ``dim``) from ``q_at``, k heads from ``k_at``
+    and v heads (``heads`` of ``vdim``) from ``v_at``; ``proj`` [tokens, columns] one number a head from ``beta_at`` and
+    ``decay_at`` on and, with ``gate_at``, a gate of heads * vdim columns.  q and k become unit vectors over a head (x /
+    sqrt(sum x^2 + unit_eps)), q times ``query_scale``; value head h uses q/k head h // (heads / key_heads).  beta =
+    sigmoid(proj), g = exp(rate softplus(proj + dt_bias)) (``rate``, not positive, and ``dt_bias`` float32 [heads]).  Per
+    request and head, token by token from the float32 ``state`` [slots, heads, dim, vdim] of the request's slot, which is
+    left as the state after the step's last token: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q.  Every
+    head's o is divided by its root mean square (``unit_norm``, with ``eps``), multiplied by ``norm_weight`` (float32
+    [vdim]) and act(gate), and rounded to the storage type: [tokens, heads * vdim].  ``raw_out`` (float32) receives o.
+
+    A step in which every entry is one token runs as one launch, a CTA a (request, head), unless ``raw_out`` asks for the
+    scan."""
+    _need_cuda(mixed, proj, rate, dt_bias, norm_weight, state, row_starts, state_slots, token_row, out, raw_out)
+    tokens = mixed.shape[0]
+    rows = _entry_checks("delta_rule", tokens, row_starts, state_slots, token_row)
+    if mixed.dim() != 2 or proj.dim() != 2 or proj.shape[0] != tokens or mixed.stride(1) != 1 or proj.stride(1) != 1 \
+            or mixed.dtype != proj.dtype:
+        raise KernelError("delta_rule: mixed and proj are [tokens, columns] of one dtype with contiguous rows")
+    if key_heads <= 0 or heads % key_heads or not 0 < dim <= DELTA_MAX_DIM or vdim <= 0:
+        raise KernelError(f"delta_rule takes whole groups of heads and key sizes up to {DELTA_MAX_DIM}, not {dim}")
+    spans = [(mixed, q_at, key_heads * dim), (mixed, k_at, key_heads * dim), (mixed, v_at, heads * vdim),
+             (proj, beta_at, heads), (proj, decay_at, heads)]
+    if gate_at is not None:
+        spans.append((proj, gate_at, heads * vdim))
+    if any(at < 0 or at + size > t.shape[1] for t, at, size in spans):
+        raise KernelError("delta_rule: the heads do not fit the rows")
+    for name, t, shape in (("rate", rate, (heads,)), ("dt_bias", dt_bias, (heads,)), ("norm_weight", norm_weight, (vdim,))):
+        if t is not None and (t.dtype != torch.float32 or t.shape != shape or not t.is_contiguous()):
+            raise KernelError(f"delta_rule: {name} must be contiguous float32 {list(shape)}")
+    if state.dtype != torch.float32 or state.dim() != 4 or state.shape[1:] != (heads, dim, vdim) or not state.is_contiguous():
+        raise KernelError("delta_rule: the state is contiguous float32 [slots, heads, dim, vdim]")
+    if gate_act not in RETENTION_ACTS:
+        raise KernelError(f"delta_rule: gate activation {gate_act!r} is not known")
+    if out is None:
+        out = torch.empty((tokens, heads * vdim), dtype=mixed.dtype, device=mixed.device)
+    elif out.shape != (tokens, heads * vdim) or out.dtype != mixed.dtype or out.stride(1) != 1:
+        raise KernelError("delta_rule: out must be [tokens, heads * vdim] of the storage type")
+    group, tag, element = heads // key_heads, dtype_tag(mixed.dtype), mixed.element_size()
+    if tokens == rows and raw_out is None and delta_step_takes(dim, vdim):
+        fn = _fn("delta_rule", "tvb_delta_step",
+                 [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p,
+                  c_void_p, c_float, c_float, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                  c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+        _check(fn(mixed.data_ptr(), mixed.stride(0), q_at, k_at, v_at, proj.data_ptr(), proj.stride(0), beta_at, decay_at,
+                  -1 if gate_at is None else gate_at, RETENTION_ACTS[gate_act], rate.data_ptr(), dt_bias.data_ptr(),
+                  query_scale, unit_eps, _ptr(norm_weight), 1 if unit_norm else 0, eps, state.data_ptr(),
+                  row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(), out.data_ptr(), out.stride(0), rows,
+                  heads, group, dim, vdim, tag, _stream()), "delta_step")
+        return out
+    if raw_out is None:
+        raw_out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=mixed.device)
+    elif raw_out.shape != (tokens, heads * vdim) or raw_out.dtype != torch.float32 or not raw_out.is_contiguous():
+        raise KernelError("delta_rule: raw_out must be contiguous float32 [tokens, heads * vdim]")
+    padded = -(-dim // 4) * 4
+    vectors = torch.empty((2, tokens, key_heads, padded), dtype=torch.float32, device=mixed.device)
+    scalars = torch.empty((tokens, heads, 4), dtype=torch.float32, device=mixed.device)
+    fn = _fn("delta_rule", "tvb_delta_prepare",
+             [c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
+              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(mixed.data_ptr(), mixed.stride(0), q_at, k_at, proj.data_ptr(), proj.stride(0), beta_at, decay_at,
+              rate.data_ptr(), dt_bias.data_ptr(), query_scale, unit_eps, vectors[0].data_ptr(), vectors[1].data_ptr(),
+              scalars.data_ptr(), tokens, key_heads, group, dim, padded, tag, _stream()), "delta_prepare")
+    fn = _fn("delta_rule", "tvb_delta_scan",
+             [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+              c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(vectors[0].data_ptr(), vectors[1].data_ptr(), scalars.data_ptr(), mixed.data_ptr() + v_at * element,
+              mixed.stride(0), state.data_ptr(), row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(),
+              raw_out.data_ptr(), rows, heads, group, dim, padded, vdim, tag, _stream()), "delta_scan")
+    finish = _fn_of("retention", "tvb_retention_finish", _RETENTION_FINISH_ARGS)
+    gate_ptr = None if gate_at is None else proj.data_ptr() + gate_at * element
+    _check(finish(raw_out.data_ptr(), gate_ptr, proj.stride(0), out.data_ptr(), out.stride(0), tokens, heads, vdim,
+                  1 if unit_norm else 0, eps, RETENTION_ACTS[gate_act if gate_at is not None else None],
+                  _ptr(norm_weight), tag, _stream()), "delta_finish")
     return out
 
 

@@ -1,7 +1,7 @@
 """The parts a model is put together from, and their registries."""
 
-from . import (attention, block, embedding, hyper, mlp, norm, parallel, retention, rope,  # noqa: F401  (they
-               selective_scan)                                                           # register themselves)
+from . import (attention, block, delta_rule, embedding, hyper, mlp, norm, parallel,  # noqa: F401  (they
+               recurrent_unit, retention, rope, selective_scan)                     # register themselves)
 from .base import Block, BuildContext, KVNeed, ParamSource, ParamSpec, Part, StateNeed
 from .registry import build_part, part_kinds, register_part
 

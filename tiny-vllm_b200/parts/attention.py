@@ -143,6 +143,9 @@ class WindowedAttention(Part):
     added before a value is cached, the second behind the output product (a host that norms the output adds it
     itself: ``output_bias``).  ``softcap``: a scaled score s becomes softcap * tanh(s / softcap).
 
+    ``reads_other_cache``: the mixer has no key and value projections; its runs read the cache of an earlier run (the
+    run list's ``cache_from``), with queries, window and everything else of their own.
+
     ``hosted=True``: a block computes the input projections of all its parts as one product and
     the output projections as another; the mixer then owns no matrices, names its share
     (``input_rows``, ``output_cols``) and works between the two products (``between``)."""
@@ -156,9 +159,12 @@ class WindowedAttention(Part):
                  sink: bool | float = False, float32_output: bool = False, qk_bias: bool = False,
                  values_are_keys: bool = False, distance_table: tuple | None = None,
                  segment: int | None = None, v_bias: bool = False, o_bias: bool = False,
-                 softcap: float | None = None) -> None:
+                 softcap: float | None = None, reads_other_cache: bool = False) -> None:
         if num_heads % num_kv_heads:
             raise ValueError("query heads must be a multiple of key-value heads")
+        if reads_other_cache and (qk_bias or v_bias or values_are_keys or value_mix is not None or qk_norm == "whole"):
+            raise ValueError("a mixer that reads another run's keys and values makes none of its own")
+        self.reads_other_cache = bool(reads_other_cache)
         limit = kernels.ATTENTION_ROWS_MAX_DIM
         if not 0 < key_dim <= limit or not 0 < value_dim <= limit:
             raise ValueError(f"the attention kernels take key and value sizes up to {limit}, not {key_dim} / {value_dim}")
@@ -229,12 +235,12 @@ class WindowedAttention(Part):
 
     @property
     def k_cols(self) -> int:
-        return self.num_kv_heads * self.key_dim
+        return 0 if self.reads_other_cache else self.num_kv_heads * self.key_dim
 
     @property
     def v_cols(self) -> int:
-        """Columns of the value projection (none when the values are the keys)."""
-        return 0 if self.values_are_keys else self.num_kv_heads * self.value_dim
+        """Columns of the value projection (none when the values are the keys, or another run's)."""
+        return 0 if self.values_are_keys or self.reads_other_cache else self.num_kv_heads * self.value_dim
 
     @property
     def out_cols(self) -> int:
@@ -254,8 +260,10 @@ class WindowedAttention(Part):
     def input_rows(self):
         """(checkpoint tensor, rows) of the input projections, in the order of their columns:
         q heads, k heads, v heads and, with a gate, the gate."""
-        rows = [(self.names["q"], self.q_cols), (self.names["k"], self.k_cols)]
-        if not self.values_are_keys:
+        rows = [(self.names["q"], self.q_cols)]
+        if not self.reads_other_cache:
+            rows.append((self.names["k"], self.k_cols))
+        if self.v_cols:
             rows.append((self.names["v"], self.v_cols))
         if self.gate:
             rows.append((self.names["g"], self.gate_cols))
@@ -273,10 +281,11 @@ class WindowedAttention(Part):
             # every layer that takes part stores the scalar; the one that hands its values on ignores it
             specs.append(ParamSpec.scalar("vmix", self.names["vmix"]))
         if self.qk_norm == "weight":
-            specs += [ParamSpec.single("q_norm_weight", self.names["q_norm"], (self.key_dim,),
-                                       role="vector", init="around_one"),
-                      ParamSpec.single("k_norm_weight", self.names["k_norm"], (self.key_dim,),
-                                       role="vector", init="around_one")]
+            specs.append(ParamSpec.single("q_norm_weight", self.names["q_norm"], (self.key_dim,),
+                                          role="vector", init="around_one"))
+            if not self.reads_other_cache:
+                specs.append(ParamSpec.single("k_norm_weight", self.names["k_norm"], (self.key_dim,),
+                                              role="vector", init="around_one"))
         if self.qk_norm == "whole":
             specs += [ParamSpec.single("q_norm_weight", self.names["q_norm"], (self.q_cols,),
                                        role="vector", init="around_one"),

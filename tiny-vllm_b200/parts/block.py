@@ -237,7 +237,56 @@ class SandwichResidualBlock(Block):
         return None, stream
 
 
+class OutputNormResidualBlock(Block):
+    """A norm behind every sublayer and none in front: x <- x + norm1(mixer(x)), then, where the layer has a
+    feed-forward, x <- x + norm2(feed_forward(x)); both sublayers read x itself.  The stream x is float32 whatever the
+    storage type; the norms hand on, beside it, its one rounding to the storage type, which is what the next products
+    read.  A checkpoint may hold the second norm of a layer without a feed-forward; nothing reads it.
+
+    The norm behind a sublayer, the residual sum and the rounding run as one kernel (``norm.after``); what the block's
+    last sublayer leaves is handed on as ``stream.pending``, which the next block, or the model's last norm, adds in a
+    pass of its own.  The block returns (None, stream)."""
+
+    def __init__(self, ctx: BuildContext, *, mixer, feed_forward, norm, mixer_norm_name: str,
+                 feed_forward_norm_name: str, mixer_name: str, feed_forward_name: str) -> None:
+        def build_norm(name, **more):
+            return ctx.build("norm", norm.with_params(name=f"{ctx.prefix}.{name}", **more), ctx)
+
+        self.mixer_norm = build_norm(mixer_norm_name)
+        self.mixer = ctx.build("mixer", mixer, ctx.child(mixer_name))
+        self.feed_forward_norm = build_norm(feed_forward_norm_name, **({"optional": True} if feed_forward is None else {}))
+        self.feed_forward = None
+        if feed_forward is not None:
+            self.feed_forward = ctx.build("feed_forward", feed_forward, ctx.child(feed_forward_name))
+        if not hasattr(self.mixer_norm, "after") or not hasattr(self.mixer_norm, "settle"):
+            raise ValueError("a block with norms behind its sublayers needs norms that offer after() and settle()")
+
+    def children(self):
+        return [part for part in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
+                if part is not None]
+
+    def forward(self, hidden, residual, ctx, run: int):
+        from .norm import PendingUpdate
+
+        if residual is None:                 # the first block: a float32 embedding starts the stream
+            stream, x = hidden, getattr(hidden, "rounded", None)
+            if x is None:
+                x, stream = self.mixer_norm.settle(stream)
+        else:
+            if hidden is not None:
+                raise ValueError("a block with norms behind its sublayers follows blocks that leave nothing but the stream")
+            x, stream = self.mixer_norm.settle(residual)
+        mixed = self.mixer.forward(x, ctx, run)
+        if self.feed_forward is None:
+            stream.pending = PendingUpdate(mixed, self.mixer_norm)
+            return None, stream
+        x, stream = self.mixer_norm.after(stream, mixed, rounded=True)
+        stream.pending = PendingUpdate(self.feed_forward.forward(x, ctx), self.feed_forward_norm)
+        return None, stream
+
+
 register_part("block", "prenorm_residual", PreNormResidualBlock)
+register_part("block", "output_norm_residual", OutputNormResidualBlock)
 register_part("block", "sandwich_residual", SandwichResidualBlock)
 register_part("block", "postnorm_residual", PostNormResidualBlock)
 register_part("block", "parallel_residual", ParallelResidualBlock)

@@ -15,10 +15,15 @@ from .registry import register_part
 
 class TokenEmbedding(Part):
     """h = E[ids]; with ``norm`` (a norm part that offers ``start``) the rows are normed at once and leave
-    in float32, as the first tensor of a float32 residual stream."""
+    in float32, as the first tensor of a float32 residual stream.  With ``stream_scale`` they are multiplied by it in
+    float32 and start the stream as they are; the rows rounded to the storage type ride on it as ``rounded``."""
 
-    def __init__(self, ctx: BuildContext, *, vocab_size: int, width: int, name: str, norm=None) -> None:
+    def __init__(self, ctx: BuildContext, *, vocab_size: int, width: int, name: str, norm=None,
+                 stream_scale: float | None = None) -> None:
+        if norm is not None and stream_scale is not None:
+            raise ValueError("an embedding is normed or scaled")
         self.vocab_size, self.width, self.name = vocab_size, width, name
+        self.stream_scale = None if stream_scale is None else float(stream_scale)
         self.weight = None
         self.norm = ctx.build("norm", norm, ctx) if norm is not None else None
         if self.norm is not None and not hasattr(self.norm, "start"):
@@ -31,6 +36,10 @@ class TokenEmbedding(Part):
         return [self.norm] if self.norm is not None else []
 
     def forward(self, token_ids):
+        if self.stream_scale is not None:
+            stream, rounded = kernels.embed_scaled(self.weight, token_ids, self.stream_scale)
+            stream.rounded = rounded
+            return stream
         rows = kernels.embed_rows(self.weight, token_ids)
         return rows if self.norm is None else self.norm.start(rows)
 

@@ -223,12 +223,15 @@ register_part("feed_forward", "gated_routed_experts", GatedRoutedExperts)
 
 class SoftmaxRoutedExperts(Part):
     """A mixture of gated experts, down_e(silu(gate_e h) * (up_e h)), routed by a softmax over all slots, some of
-    which may hand their input on unchanged.
+    which may hand their input on unchanged.  With ``limit`` an expert is g = min(gate_e h, limit), u = clamp(up_e h,
+    -limit, limit), y = g * sigmoid(alpha * g) * (u + 1) instead.
 
     Router logits z = W_router h are float32 and have ``experts + identity`` entries; the scores are s =
     softmax(z) over all of them.  A token uses the ``top`` slots with the largest choice scores s + correction
     (tensor ``correction``, with ``correction=True``; the weights use s without it), weighted by s as it is
-    (``renormalise``: divided by the sum of the chosen scores).  The last ``identity`` slots are experts without
+    (``renormalise``: divided by the sum of the chosen scores).  With ``groups`` > 1 the slots form that many equal
+    groups of neighbours, a group's score is its largest choice score, and only slots of the ``keep`` best groups can
+    be chosen.  The last ``identity`` slots are experts without
     tensors whose output is h itself.
 
     As in :class:`RoutedExperts` the experts are two products: [gate_e | up_e] of all experts are the rows of
@@ -239,7 +242,16 @@ class SoftmaxRoutedExperts(Part):
 
     def __init__(self, ctx: BuildContext, *, hidden_size: int, experts: int, top: int, ff: int, identity: int = 0,
                  correction: bool = False, renormalise: bool = False, float32_output: bool = False,
-                 names: dict | None = None) -> None:
+                 names: dict | None = None, groups: int = 1, keep: int = 1, limit: float | None = None,
+                 alpha: float = 1.0) -> None:
+        if groups <= 0 or (experts + identity) % groups or not 0 < keep <= groups:
+            raise ValueError("slots form equal groups of which at least one and at most all are kept")
+        if top > (experts + identity) // groups * keep:
+            raise ValueError("the groups that are kept hold fewer slots than a token uses")
+        if limit is not None and not limit > 0:
+            raise ValueError("a limit on an expert's activations is positive")
+        self.groups, self.keep = groups, keep
+        self.limit, self.alpha = None if limit is None else float(limit), float(alpha)
         if experts <= 0 or identity < 0 or experts + identity > kernels.ROUTE_MAX_EXPERTS or not 0 < top <= experts + identity:
             raise ValueError(f"a token uses between 1 and all of at most {kernels.ROUTE_MAX_EXPERTS} slots")
         self.hidden_size, self.experts, self.identity, self.top, self.ff = hidden_size, experts, identity, top, ff
@@ -279,7 +291,8 @@ class SoftmaxRoutedExperts(Part):
         logits = linear(x, self.router_weight, out_dtype=torch.float32)
         inner, passed = kernels.route_softmax_gated(
             logits, linear(x, self.in_weight), experts=self.experts, identity=self.identity, top=self.top,
-            ff=self.ff, correction=self.correction, renormalise=self.renormalise)
+            ff=self.ff, correction=self.correction, renormalise=self.renormalise, groups=self.groups, keep=self.keep,
+            limit=self.limit, alpha=self.alpha)
         return linear(inner, self.down_weight, out_dtype=self.out_dtype), passed
 
     def forward(self, x, ctx):

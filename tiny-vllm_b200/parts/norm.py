@@ -58,8 +58,9 @@ class StreamRMSNorm(Part):
     also where activations and weights are bfloat16."""
 
     def __init__(self, ctx: BuildContext, *, width: int, eps: float, name: str | None = None,
-                 unit_offset: bool = False) -> None:
+                 unit_offset: bool = False, optional: bool = False) -> None:
         self.width = width
+        self.optional = optional          # the checkpoint may lack the weight: ``weight`` stays None
         self.eps = float(eps)
         self.name = name if name is not None else f"{ctx.prefix}.weight"
         self.out_dtype = ctx.dtype
@@ -68,7 +69,7 @@ class StreamRMSNorm(Part):
 
     def param_specs(self):
         return [ParamSpec.single("weight", self.name, (self.width,), role="vector",
-                                 init="normal" if self.unit_offset else "around_one")]
+                                 init="normal" if self.unit_offset else "around_one", optional=self.optional)]
 
     def finalize(self) -> None:
         if self.unit_offset and self.weight is not None and not getattr(self, "_offset_applied", False):
@@ -103,9 +104,29 @@ class StreamRMSNorm(Part):
             stream.pending = None
         return out, updated
 
-    def after(self, stream, y, following=None, row_scale=None, x=None):
+    def settle(self, stream):
+        """(s' rounded to the storage type, s') with s' = stream + what is pending on it, in one pass; in the float32
+        path the two are one tensor."""
+        pending = getattr(stream, "pending", None)
+        if pending is None and stream.dtype == self.out_dtype:
+            return stream, stream
+        pending = pending or PendingUpdate(None)
+        post = pending.norm
+        rounded, stream = kernels.sandwich_norm(
+            stream, pending.y, post_weight=None if post is None else post.weight,
+            post_eps=0.0 if post is None else post.eps, row_scale=pending.row_scale, x=pending.x,
+            out_dtype=self.out_dtype, rounded=self.out_dtype != stream.dtype)
+        stream.pending = None
+        return (stream if rounded is None else rounded), stream
+
+    def after(self, stream, y, following=None, row_scale=None, x=None, rounded: bool = False):
         """This norm behind a sublayer: (following(s'), s') with s' = stream + norm(y + row_scale * x), the stream
-        updated in place; ``following`` is the norm in front of the next sublayer (None: no first result)."""
+        updated in place; ``following`` is the norm in front of the next sublayer (None: no first result, or, with
+        ``rounded``, s' rounded to the storage type; in the float32 path that is the stream itself)."""
+        if rounded:
+            out, stream = kernels.sandwich_norm(stream, y, post_weight=self.weight, post_eps=self.eps, row_scale=row_scale,
+                                                x=x, out_dtype=self.out_dtype, rounded=self.out_dtype != stream.dtype)
+            return (stream if out is None else out), stream
         return kernels.sandwich_norm(
             stream, y, post_weight=self.weight, post_eps=self.eps,
             pre_weight=None if following is None else following.weight,
