@@ -22,9 +22,10 @@
 
 __device__ __forceinline__ float delta_softplus(float z) { return __fadd_rn(fmaxf(z, 0.0f), log1pf(expf(-fabsf(z)))); }
 __device__ __forceinline__ float delta_sigmoid(float z) { return __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z))); }
-// exp(rate softplus(a + bias)), rate = -exp(A_log)
+// exp(rate softplus(a + bias)), rate = -exp(A_log); taken as 1 + (exp(x) - 1): a head that keeps hundreds of tokens
+// multiplies it hundreds of times, and an exponential that is one unit off to one side there would show
 __device__ __forceinline__ float delta_decay(float a, float bias, float rate) {
-    return expf(__fmul_rn(rate, delta_softplus(__fadd_rn(a, bias))));
+    return __fadd_rn(1.0f, expm1f(__fmul_rn(rate, delta_softplus(__fadd_rn(a, bias)))));
 }
 
 // two float32 numbers in one 64-bit register: the arithmetic unit's two-wide forms

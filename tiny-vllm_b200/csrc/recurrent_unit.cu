@@ -22,27 +22,27 @@
 #define UNIT_LOG2E 1.4426950408889634f
 
 // The unit's float32 functions.  With 16-bit storage they take the special-function unit's 2^x, 1 / x and root (a few
-// units in the last place, far below the rounding of what goes in).
-//   decay     exp(x)
-//   written   sqrt(1 - exp(2 x)) for x <= 0
+// units in the last place, far below the rounding of what goes in).  Both the decay a = 1 + e and what is written,
+// sqrt(1 - a^2) = sqrt(-e (2 + e)), come from e = exp(x) - 1, x <= 0: a channel that keeps hundreds of tokens multiplies
+// a hundreds of times, and an exponential that is one unit off to one side there would show.
 template <typename T> struct Unit;
 template <> struct Unit<float> {
     static __device__ __forceinline__ float sigmoid(float z) { return __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-z))); }
-    static __device__ __forceinline__ float decay(float x) { return expf(x); }
-    static __device__ __forceinline__ float written(float x) { return __fsqrt_rn(fmaxf(-expm1f(__fmul_rn(2.0f, x)), 0.0f)); }
+    static __device__ __forceinline__ float lost(float x) { return expm1f(x); }
+    static __device__ __forceinline__ float root(float x) { return __fsqrt_rn(x); }
 };
 template <> struct Unit<bf16> {
     static __device__ __forceinline__ float sigmoid(float z) {
         return reciprocal_unit(1.0f + exp2_unit(__fmul_rn(-z, UNIT_LOG2E)));
     }
-    static __device__ __forceinline__ float decay(float x) { return exp2_unit(__fmul_rn(x, UNIT_LOG2E)); }
-    static __device__ __forceinline__ float written(float x) {
-        const float z = __fmul_rn(-2.0f, x);      // 1 - exp(-z): by its series where the difference would cancel
-        const float series = z * __fmaf_rn(z, __fmaf_rn(z, __fmaf_rn(z, -0.041666668f, 0.16666667f), -0.5f), 1.0f);
-        const float plain = 1.0f - exp2_unit(__fmul_rn(-z, UNIT_LOG2E));
-        float root;
-        asm("sqrt.approx.ftz.f32 %0, %1;\n" : "=f"(root) : "f"(z < 0.0625f ? series : plain));
-        return root;
+    static __device__ __forceinline__ float lost(float x) {       // by its series where the difference would cancel
+        const float series = x * __fmaf_rn(x, __fmaf_rn(x, __fmaf_rn(x, 0.041666668f, 0.16666667f), 0.5f), 1.0f);
+        return x > -0.0625f ? series : exp2_unit(__fmul_rn(x, UNIT_LOG2E)) - 1.0f;
+    }
+    static __device__ __forceinline__ float root(float x) {
+        float y;
+        asm("sqrt.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+        return y;
     }
 };
 
@@ -67,9 +67,10 @@ struct UnitArgs {
 // Decay and new input of one channel at one token.
 template <typename T> __device__ __forceinline__ void unit_terms(float pre_r, float pre_i, float u, float br, float bi,
                                                                  float c, float& a, float& b) {
-    const float x = __fmul_rn(c, Unit<T>::sigmoid(__fadd_rn(pre_r, br)));
-    a = Unit<T>::decay(x);
-    b = __fmul_rn(__fmul_rn(Unit<T>::written(x), Unit<T>::sigmoid(__fadd_rn(pre_i, bi))), u);
+    const float e = Unit<T>::lost(__fmul_rn(c, Unit<T>::sigmoid(__fadd_rn(pre_r, br))));
+    a = __fadd_rn(1.0f, e);
+    const float written = Unit<T>::root(fmaxf(__fmul_rn(-e, __fadd_rn(2.0f, e)), 0.0f));
+    b = __fmul_rn(__fmul_rn(written, Unit<T>::sigmoid(__fadd_rn(pre_i, bi))), u);
 }
 
 template <typename T>
