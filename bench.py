@@ -1615,38 +1615,13 @@ def zifunex_workload(args) -> int:
     every layer: tokens/s through the engine, and every kernel of both designs with the fraction of its roofline.
     One JSON line."""
     layers = args.layers if args.layers_given else 6
-    batch, prompt, steps, warmup = args.batch, PROMPT_TOKENS, min(args.steps, 64), max(args.warmup, 3)
+    batch, prompt = args.batch, PROMPT_TOKENS
     peak, peak_source = peaks()
     names = ("hyper_norm", "stream_norm", "qkv_prepare", "attention_tiles", "attention_tiles_singles", "attention_rows",
              "gated_recurrence", "retention", "selective_scan", "short_convolution", "gated_act", "embed_pairs")
-    results = []
-    sampler = ClockSampler()
-    sampler.start()
-    sizes = [size for size in KELASUN_SIZES if not args.sizes or size in args.sizes.split(",")]
-    for size in sizes:
-        row = {"size": size}
-        for label, config in (("zifunex", zifunex_config(size, layers)), ("bimolix", dense_bimolix_config(size, layers))):
-            decode, prefill_ms, by_prompt, by_decode, weight_bytes = measure_design(
-                config, names, batch, prompt, steps, warmup, sampler)
-            kernels_out = {}
-            for phase, marks, tokens in (("prefill", by_prompt, prompt), ("decode", by_decode, batch)):
-                found = {}
-                for name, start, end in marks:
-                    calls, ms = found.get(name, (0, 0.0))
-                    found[name] = (calls + 1, ms + start.elapsed_time(end))
-                for name, (calls, ms) in sorted(found.items()):
-                    per_call = 1e3 * ms / calls
-                    roofline = zifunex_roofline if label == "zifunex" else bimolix_roofline
-                    ideal, bound = roofline(name, size, tokens, prompt, peak)
-                    kernels_out[f"{phase}:{name}"] = {
-                        "calls": calls, "us_per_call": round(per_call, 2), "roofline_us": round(ideal, 2),
-                        "bound": bound, "frac": round(ideal / per_call, 3) if per_call > 0 else None}
-            row[label] = {
-                "decode_tokens_per_s": round(decode["tokens_per_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
-                "prefill_tokens_per_s": round(prompt / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
-                "weight_bytes": weight_bytes, "kernels": kernels_out}
-        results.append(row)
-    sampler.stop()
+    sizes, results, clocks = designs_side_by_side(args, names, peak, {
+        "zifunex": (lambda size: zifunex_config(size, layers), zifunex_roofline),
+        "bimolix": (lambda size: dense_bimolix_config(size, layers), bimolix_roofline)})
     print(json.dumps({
         "metric": "Zifunex beside Bimolix of equal layer sizes: decode tok/s at batch "
                   f"{batch} from context {prompt:,}, prefill tok/s of {prompt:,} tokens, bf16",
@@ -1661,7 +1636,152 @@ def zifunex_workload(args) -> int:
         "peaks": {"hbm_gbs": peak["hbm_gbs"], "bf16_tflops": peak["bf16_tflops"],
                   "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1), "exp_per_s_nominal": EXP_RATE_NOMINAL,
                   "source": peak_source},
-        "clocks": sampler.summary(), "results": results}))
+        "clocks": clocks, "results": results}))
+    return 0
+
+
+def designs_side_by_side(args, names, peak: dict, designs: dict):
+    """Every size's designs (label -> (size -> configuration, roofline)) measured one after the other with
+    :func:`measure_design`: (sizes, a row a size, clocks seen)."""
+    batch, prompt, steps, warmup = args.batch, PROMPT_TOKENS, min(args.steps, 64), max(args.warmup, 3)
+    results = []
+    sampler = ClockSampler()
+    sampler.start()
+    sizes = [size for size in KELASUN_SIZES if not args.sizes or size in args.sizes.split(",")]
+    for size in sizes:
+        row = {"size": size}
+        for label, (config_of, roofline) in designs.items():
+            config = config_of(size)
+            decode, prefill_ms, by_prompt, by_decode, weight_bytes = measure_design(
+                config, names, batch, prompt, steps, warmup, sampler)
+            kernels_out = {}
+            for phase, marks, tokens in (("prefill", by_prompt, prompt), ("decode", by_decode, batch)):
+                found = {}
+                for name, start, end in marks:
+                    calls, ms = found.get(name, (0, 0.0))
+                    found[name] = (calls + 1, ms + start.elapsed_time(end))
+                for name, (calls, ms) in sorted(found.items()):
+                    per_call = 1e3 * ms / calls
+                    ideal, bound = roofline(name, size, tokens, prompt, peak)
+                    kernels_out[f"{phase}:{name}"] = {
+                        "calls": calls, "us_per_call": round(per_call, 2), "roofline_us": round(ideal, 2),
+                        "bound": bound, "frac": round(ideal / per_call, 3) if per_call > 0 else None}
+            row[label] = {
+                "decode_tokens_per_s": round(decode["tokens_per_s"], 1), "decode_ms_per_step": round(decode["ms_per_step"], 4),
+                "prefill_tokens_per_s": round(prompt / (prefill_ms / 1e3), 1), "prefill_ms": round(prefill_ms, 3),
+                "weight_bytes": weight_bytes, "kernels": kernels_out}
+        results.append(row)
+    sampler.stop()
+    return sizes, results, sampler.summary()
+
+
+# ------------------------------------------- Lasupel beside Bimolix at equal layer sizes
+LASUPEL_WINDOW, LASUPEL_TAPS = 1024, 4
+# (kernel of the new design, its counterpart in Bimolix) by what they do
+LASUPEL_LIKE = (
+    ("sandwich_norm", "stream_norm", "norm + residual sum"),
+    ("qkv_prepare", "qkv_prepare", "q/k norm, rotation or bias, cache write"),
+    ("attention_tiles", "attention_tiles", "prompt attention"),
+    ("attention_tiles_singles", "attention_tiles_singles", "decode attention"),
+    ("delta_rule", "retention", "linear attention"),
+    ("recurrent_unit", "retention", "the other recurrence"),
+    ("block_products", None, "the recurrent unit's gates (a library product)"),
+    ("short_convolution", "gated_act", "a pass over the activations"),
+    ("route_softmax_gated", "route_gated_act", "routing + activation"),
+    ("gated_act", "gated_act", "act(gate) * up"),
+)
+
+
+def lasupel_config(size: str, layers: int):
+    """A recurrent unit as wide as the model, attention over a window of 1,024 keys, a delta rule with two value heads a
+    key head, and attention that reads the keys of the layer two before, in turn; recurrent layers with a dense
+    feed-forward, attention layers with experts as many and as wide as Bimolix's at this size."""
+    from tinyvllm_b200.models import LasupelConfig
+    from tinyvllm_b200.models.lasupel import (LasupelAttention, LasupelDelta, LasupelFeedForward, LasupelLayer,
+                                              LasupelRecurrentUnit)
+
+    width, heads, kv, dim, ff = KELASUN_SIZES[size]
+    dense = LasupelFeedForward(kind="dense", ff=ff)
+    experts = LasupelFeedForward(kind="moe", ff=kelasun_expert_width(ff), limit=7.0, experts=KELASUN_EXPERTS, top=KELASUN_TOP,
+                                 groups=4, keep=2)
+    made = []
+    for index in range(layers):
+        attention = LasupelAttention(heads=heads, kv_heads=kv, dim=dim, vdim=dim, scale=dim ** -0.5, window=LASUPEL_WINDOW,
+                                     rot_dims=dim // 2, rot_base=1000000.0, kv_from=index - 2 if index % 4 == 3 else None)
+        if index % 2 == 1:
+            made.append(LasupelLayer(attention, experts))
+        elif index % 4 == 0:
+            made.append(LasupelLayer(LasupelRecurrentUnit(width=width, blocks=heads, conv=LASUPEL_TAPS), dense))
+        else:
+            made.append(LasupelLayer(LasupelDelta(heads=heads, kv_heads=heads // 2, dim=dim, vdim=dim, conv=LASUPEL_TAPS), dense))
+    return LasupelConfig(vocab=MODEL["vocab_size"], width=width, norm_eps=1e-6, embedding_scale=width ** 0.5, layers=tuple(made))
+
+
+def lasupel_roofline(name: str, size: str, tokens: int, context: int, peak: dict):
+    """(microseconds at the peaks, what bounds it) of one call of kernel ``name`` in a Lasupel layer: ``tokens``
+    new tokens whose requests hold ``context`` tokens each (a prompt: context == tokens)."""
+    width, heads, kv, dim, ff = KELASUN_SIZES[size]
+    prompt, part = context == tokens, width // heads
+    seen = lambda p: min(p + 1, LASUPEL_WINDOW)                       # keys the query at position p attends
+    bytes_, limits = 0.0, []
+    if name == "sandwich_norm":
+        bytes_ = tokens * width * (4 + 4 + 4 + 2)
+    elif name == "qkv_prepare":
+        # q in place in every attention layer; k and v to their pages in every other one
+        bytes_ = tokens * dim * 2 * (2 * heads + 4 * kv / 2)
+    elif name == "attention_tiles":
+        limits.append((2.0 * heads * 2 * dim * sum(seen(p) for p in range(tokens)) / (peak["bf16_tflops"] * 1e12), "tensor"))
+    elif name == "attention_tiles_singles":
+        bytes_ = tokens * kv * seen(context) * 2 * dim * 2
+    elif name == "short_convolution":                                 # of the unit and of the delta rule in turn
+        bytes_ = tokens * (width + 2 * heads * dim) / 2 * (2 * 2 + (0 if prompt else (LASUPEL_TAPS - 1) * 4 * 2))
+    elif name == "recurrent_unit":
+        bytes_ = tokens * width * (2 + 2 + 2 + (8 if prompt else 4 * 2)) + (0 if prompt else 2 * width * part * 2)
+    elif name == "block_products":
+        bytes_ = tokens * width * (2 + 8) + 2 * width * part * 2
+        limits.append((2.0 * tokens * width * 2 * part / (peak["bf16_tflops"] * 1e12), "tensor"))
+    elif name == "delta_rule":
+        # read under the key, write, read-out: a multiply-add each
+        limits.append((6.0 * tokens * heads * dim * dim / (FP32_TFLOPS_NOMINAL * 1e12), "fp32 (nominal)"))
+        bytes_ = (0 if prompt else tokens) * heads * dim * dim * 4 * 2 + tokens * heads * dim * 2 * 4
+    elif name == "route_softmax_gated":
+        bytes_ = tokens * KELASUN_EXPERTS * kelasun_expert_width(ff) * 2 * 3
+    elif name == "gated_act":
+        bytes_ = tokens * ff * 2 * 3
+    elif name == "embed_scaled":
+        bytes_ = tokens * width * (2 + 4 + 2)
+    limits.append((bytes_ / (peak["hbm_gbs"] * 1e9), "memory"))
+    seconds, bound = max(limits)
+    return seconds * 1e6, bound
+
+
+def lasupel_workload(args) -> int:
+    """Prefill and decode of Lasupel at the layer sizes of the 0.6B, 8B and 32B models (random weights,
+    ``--layers`` layers, default 4) beside Bimolix of the same sizes, depth and feed-forwards: tokens/s through the
+    engine, and every kernel of both designs with the fraction of its roofline.  One JSON line."""
+    layers = args.layers if args.layers_given else 4
+    batch, prompt = args.batch, PROMPT_TOKENS
+    peak, peak_source = peaks()
+    names = ("sandwich_norm", "stream_norm", "qkv_prepare", "attention_tiles", "attention_tiles_singles", "attention_rows",
+             "delta_rule", "retention", "recurrent_unit", "block_products", "short_convolution", "route_softmax_gated",
+             "route_gated_act", "gated_act", "embed_scaled")
+    sizes, results, clocks = designs_side_by_side(args, names, peak, {
+        "lasupel": (lambda size: lasupel_config(size, layers), lasupel_roofline),
+        "bimolix": (lambda size: bimolix_config(size, layers), bimolix_roofline)})
+    print(json.dumps({
+        "metric": "Lasupel beside Bimolix of equal layer sizes: decode tok/s at batch "
+                  f"{batch} from context {prompt:,}, prefill tok/s of {prompt:,} tokens, bf16",
+        "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic (random weights and tokens)",
+        "config": {"layers": layers, "batch": batch, "vocab": MODEL["vocab_size"],
+                   "sizes": {k: list(v) for k, v in KELASUN_SIZES.items() if k in sizes},
+                   "window": LASUPEL_WINDOW, "taps": LASUPEL_TAPS, "experts": KELASUN_EXPERTS, "top": KELASUN_TOP,
+                   "like_kernels": [list(pair) for pair in LASUPEL_LIKE],
+                   "timing": "CUDA events; decode replays graphs with inputs uploaded every step, for "
+                             f"{batch} requests; kernel figures: the calls of one eager step queued behind a spin kernel, "
+                             "so that each pair of events brackets device time (warm caches)"},
+        "peaks": {"hbm_gbs": peak["hbm_gbs"], "bf16_tflops": peak["bf16_tflops"],
+                  "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1), "source": peak_source},
+        "clocks": clocks, "results": results}))
     return 0
 
 
@@ -1720,15 +1840,15 @@ def main() -> int:
     parser.add_argument("--warmup", type=int, default=8)
     parser.add_argument("--impl", choices=("ours", "reference"), default="ours")
     parser.add_argument("--workload", choices=("0.6b", "8b", "32b", "arrivals", "gumapel", "kelasun", "bimolix", "fezavik",
-                                               "zifunex"),
+                                               "zifunex", "lasupel"),
                         default="0.6b",
                         help="0.6b: the decode and prefill measurement (default); 8b, 32b: the serving "
                              "workloads of those sizes at full depth; arrivals: 16 requests 20 ms apart; "
                              "gumapel: the Gumapel design beside a windowed Qwen3 at equal layer sizes; "
                              "kelasun: the Kelasun design beside a dense Qwen3 at equal layer sizes; "
                              "bimolix: the Bimolix design beside Kelasun at equal layer sizes; "
-                             "fezavik, zifunex: those designs beside Bimolix at equal layer sizes")
-    parser.add_argument("--sizes", default="", help="kelasun, bimolix, fezavik, zifunex: which of 0.6b,8b,32b (default: all)")
+                             "fezavik, zifunex, lasupel: those designs beside Bimolix at equal layer sizes")
+    parser.add_argument("--sizes", default="", help="kelasun, bimolix, fezavik, zifunex, lasupel: which of 0.6b,8b,32b (default: all)")
     parser.add_argument("--layers", type=int, default=None,
                         help="fewer layers than the configuration has (both numbers are in the line)")
     parser.add_argument("--batch", type=int, default=8)
@@ -1761,6 +1881,8 @@ def main() -> int:
         return fezavik_workload(args)
     if args.workload == "zifunex":
         return zifunex_workload(args)
+    if args.workload == "lasupel":
+        return lasupel_workload(args)
     if args.eager_profile:
         return eager_profile(args, warmup)
     return headline(args, warmup)

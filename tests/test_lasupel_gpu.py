@@ -216,6 +216,42 @@ def test_recurrent_unit_from_a_carried_state(blocks, size, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+def test_slow_channels_do_not_drift(dtype):
+    """Channels that lose a thousandth to a ten-thousandth a token over 6,000 tokens: an exponential that is one unit off
+    to one side would be off by hundreds of units at the end.  So for heads of the delta rule that lose as little."""
+    from tinyvllm_b200.ops import kernels
+
+    g = torch.Generator().manual_seed(3)
+    tokens, channels = 6000, 64
+    entries, _ = entries_of([tokens], [0])
+    lam = torch.linspace(-10.0, -6.5, channels).float()
+    u, pre = torch.ones(tokens, channels), torch.zeros(tokens, 2, channels)
+    pre[:, 0] = torch.randn(tokens, channels, generator=g) * 0.3
+    zero = torch.zeros(channels)
+    decay = -8.0 * torch.nn.functional.softplus(lam.double())
+    state = torch.zeros(1, channels, device=CUDA)
+    kernels.recurrent_unit(dev(u, dtype), dev(u, dtype), blocks=1, decay=dev(decay), bias_r=dev(zero), bias_i=dev(zero),
+                           pre=dev(pre.view(tokens, 1, 2 * channels)), state=state, act=None, **entries)
+    log_a = decay.float().double() * torch.sigmoid(pre[:, 0].double())
+    assert log_a.mean(0).max() > -3e-4 and log_a.mean(0).min() < -3e-3
+    later = log_a.flip(0).cumsum(0).flip(0) - log_a                # the decays behind each token
+    want = (torch.exp(later) * torch.sqrt(-torch.expm1(2.0 * log_a)) * 0.5).sum(0)
+    close(state[0] / want.float().to(CUDA), torch.ones(channels), torch.float32, limit=2e-5 if dtype == torch.float32 else 6e-5)
+    heads, dim = 4, 8
+    rate = -torch.tensor([1e-4, 3e-4, 1e-3, 3e-3])
+    mixed, proj = torch.ones(tokens, 3 * heads * dim), torch.zeros(tokens, 2 * heads)
+    proj[:, :heads], proj[0, :heads] = -200.0, 200.0               # the first token alone writes
+    proj[:, heads:] = torch.rand(tokens, heads, generator=g)
+    proj = rounded(proj, dtype)
+    state = torch.zeros(1, heads, dim, dim, device=CUDA)
+    kernels.delta_rule(dev(mixed, dtype), dev(proj, dtype), q_at=0, k_at=heads * dim, v_at=2 * heads * dim, beta_at=0,
+                       decay_at=heads, heads=heads, key_heads=heads, dim=dim, vdim=dim, rate=dev(rate), dt_bias=dev(torch.zeros(heads)),
+                       state=state, raw_out=torch.empty(tokens, heads * dim, device=CUDA), **entries)
+    kept = torch.exp((rate.double() * plain.softplus(proj[1:, heads:])).sum(0)) / (dim + 1e-6) ** 0.5
+    close(state[0].cpu().double() / kept[:, None, None], torch.ones(heads, dim, dim), torch.float32, limit=2e-5)
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
 @pytest.mark.parametrize("heads,kv,dim,vdim", [(4, 2, 16, 32), (3, 1, 10, 7), (2, 2, 32, 48), (1, 1, 5, 3), (4, 2, 64, 128),
                                                (4, 1, 130, 24), (2, 1, 128, 128), (2, 1, 256, 40), (2, 2, 33, 256)])
 def test_delta_rule_from_a_carried_state(heads, kv, dim, vdim, dtype):
@@ -271,16 +307,18 @@ def test_delta_rule_from_a_carried_state(heads, kv, dim, vdim, dtype):
     common = dict(q_at=q_at, k_at=k_at, v_at=v_at, beta_at=beta_at, decay_at=decay_at, gate_at=gate_at, heads=heads,
                   key_heads=kv, dim=dim, vdim=vdim, rate=dev(-torch.exp(a_log)), dt_bias=dev(dt_bias), query_scale=scale,
                   unit_eps=unit_eps, norm_weight=dev(weight), eps=eps)
-    device_state = dev(state)
-    device_raw = torch.empty(starts[-1], hv, device=CUDA)
-    got = kernels.delta_rule(dev(mixed, dtype), dev(proj, dtype), state=device_state, raw_out=device_raw, **common, **entries)
-    # inputs are exact in both number formats, and all that follows them but the last rounding is float32
-    close(device_raw, raw, torch.float32, limit=1e-5)
-    close(device_state, want_state, torch.float32, limit=1e-5)
     # a norm over a head multiplies what cancelled in the head's sum: the bound is on the scale of all heads
     limit = 1e-4 if dtype == torch.float32 else None
-    close(got, want, dtype, limit=limit)
-    assert torch.equal(device_state[2].cpu(), state[2])
+    for cols in (0, 2, 4):
+        device_state = dev(state)
+        device_raw = torch.empty(starts[-1], hv, device=CUDA)
+        got = kernels.delta_rule(dev(mixed, dtype), dev(proj, dtype), state=device_state, raw_out=device_raw, cols=cols,
+                                 **common, **entries)
+        # inputs are exact in both number formats, and all that follows them but the last rounding is float32
+        close(device_raw, raw, torch.float32, limit=1e-5)
+        close(device_state, want_state, torch.float32, limit=1e-5)
+        close(got, want, dtype, limit=limit)
+        assert torch.equal(device_state[2].cpu(), state[2])
     slots = [5, 2, 7, 0, 6, 1, 3]
     entries, _ = entries_of([1] * 7, slots, padding=(3,))
     state = (torch.randn(8, heads, dim, vdim, generator=g) * 0.5).float()

@@ -4,18 +4,20 @@
 //   log a = c * r                                             c <= 0, one number a channel
 //   S <- a S + sqrt(1 - a^2) i u,    out = S act(y + b_y)     act: the tanh form of GELU, SiLU or none
 //
-//   recurrent_unit_scan   prompts: a CTA walks one entry for 32 channels, UNIT_BLOCK tokens at a time: its warps take
-//                         UNIT_RUN tokens each, side by side, leave what their tokens make of a state of zero and the
-//                         product of their decays, and walk their tokens again from the state these give them
+//   recurrent_unit_scan   prompts: a cluster of CTAs walks one entry for 32 channels, a block of UNIT_BLOCK tokens a CTA
+//                         at a time: the CTAs' warps take UNIT_RUN tokens each, side by side, leave what their tokens
+//                         make of a state of zero and the product of their decays, and walk their tokens again from the
+//                         state these give them (the CTAs read one another's sums from shared memory)
 //   recurrent_unit_step   one token a request: with `w` the gates' products are done here too (a CTA a block of gate
 //                         channels, whose weights are read once for all its requests), else the gates come as `pre`
 //
 // Gates, decays, state and sums are float32 whatever the storage type of u, y and out.
 #include "common.cuh"
 
-#define UNIT_WARPS 16
+#define UNIT_WARPS 8
 #define UNIT_RUN 8
 #define UNIT_BLOCK (UNIT_WARPS * UNIT_RUN)
+#define UNIT_MOST_CTAS 8          // of a cluster
 #define UNIT_ACT_NONE 0
 #define UNIT_ACT_SILU 1
 #define UNIT_ACT_GELU_TANH 2
@@ -73,66 +75,108 @@ template <typename T> __device__ __forceinline__ void unit_terms(float pre_r, fl
     b = __fmul_rn(__fmul_rn(written, Unit<T>::sigmoid(__fadd_rn(pre_i, bi))), u);
 }
 
+// The address in the shared memory of the cluster's CTA `rank` of what `p` is in this CTA's.
+__device__ __forceinline__ float load_of_cta(const float* p, int rank) {
+    uint32_t address;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;\n" : "=r"(address) : "r"(smem_address(p)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];\n" : "=f"(v) : "r"(address) : "memory");
+    return v;
+}
+
 template <typename T>
-__global__ void __launch_bounds__(UNIT_WARPS * 32) recurrent_unit_scan_kernel(
-    const T* __restrict__ u, const T* __restrict__ y, T* __restrict__ out, UnitArgs args) {
-    __shared__ float products[2][UNIT_WARPS][32], ends[2][UNIT_WARPS][32], carry[2][32];
-    const int row = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+__global__ void __launch_bounds__(UNIT_WARPS * 32, 3) recurrent_unit_scan_kernel(
+    const T* __restrict__ u, const T* __restrict__ y, T* __restrict__ out, UnitArgs args, int ctas) {
+    __shared__ float products[2][UNIT_WARPS][32], ends[2][UNIT_WARPS][32], block_product[2][32], block_end[2][32];
+    const int row = blockIdx.z, rank = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int begin = args.row_starts[row], count = args.row_starts[row + 1] - begin;
-    const int channel = blockIdx.x * 32 + lane;
+    const int channel = blockIdx.y * 32 + lane;
     const bool live = channel < args.channels;
-    if (count <= 0) return;
     const int at = live ? channel : 0;
-    T* dst = out + (int64_t)begin * args.out_stride + at;
-    if (args.token_row[begin] < 0) {              // a padding row of a recorded batch: no request, no state
+    const bool owned = count > 0 && args.token_row[begin] >= 0;
+    if (!owned) {                                 // the whole cluster leaves: a padding row of a recorded batch
         if (live)
-            for (int t = warp; t < count; t += UNIT_WARPS) dst[(int64_t)t * args.out_stride] = from_float<T>(0.0f);
+            for (int t = rank * UNIT_WARPS + warp; t < count; t += ctas * UNIT_WARPS)
+                out[(int64_t)(begin + t) * args.out_stride + at] = from_float<T>(0.0f);
         return;
     }
     float* mine = args.state + (int64_t)args.state_slots[row] * args.channels + at;
     const float br = args.bias_r[at], bi = args.bias_i[at], c = args.decay[at];
     const float by = args.bias_y ? args.bias_y[at] : 0.0f;
-    const T* u_in = u + (int64_t)begin * args.u_stride + at;
-    const T* y_in = y + (int64_t)begin * args.y_stride + at;
-    const float* pre_in = args.pre + (int64_t)begin * args.pre_token + (int64_t)(at / args.size) * args.pre_block + at % args.size;
-    if (warp == 0) carry[1][lane] = live ? mine[0] : 0.0f;
-    for (int first = 0, turn = 0; first < count; first += UNIT_BLOCK, turn ^= 1) {
-        const int t0 = first + warp * UNIT_RUN;
+    float carry = live ? mine[0] : 0.0f;          // the state before the cluster's tokens, in every warp
+    // this warp's first token and the pointers to it
+    int t0 = (rank * UNIT_WARPS + warp) * UNIT_RUN;
+    const T* u_in = u + (int64_t)(begin + t0) * args.u_stride + at;
+    const T* y_in = y + (int64_t)(begin + t0) * args.y_stride + at;
+    T* dst = out + (int64_t)(begin + t0) * args.out_stride + at;
+    const float* pre_in = args.pre + (int64_t)(begin + t0) * args.pre_token + (int64_t)(at / args.size) * args.pre_block + at % args.size;
+    const int step = ctas * UNIT_BLOCK;
+    for (int first = 0, turn = 0; first < count; first += step, turn ^= 1) {
         float a[UNIT_RUN], b[UNIT_RUN], pre_r[UNIT_RUN], pre_i[UNIT_RUN];
         T u_now[UNIT_RUN], y_now[UNIT_RUN];
+        const int here = live ? count - t0 : 0;   // tokens of the entry from this warp's first on
 #pragma unroll
         for (int t = 0; t < UNIT_RUN; ++t)        // all loads of a block are in flight together
-            if (live && t0 + t < count) {
-                pre_r[t] = pre_in[(int64_t)(t0 + t) * args.pre_token];
-                pre_i[t] = pre_in[(int64_t)(t0 + t) * args.pre_token + args.size];
-                u_now[t] = u_in[(int64_t)(t0 + t) * args.u_stride];
-                y_now[t] = y_in[(int64_t)(t0 + t) * args.y_stride];
+            if (t < here) {
+                pre_r[t] = pre_in[t * args.pre_token];
+                pre_i[t] = pre_in[t * args.pre_token + args.size];
+                u_now[t] = u_in[t * args.u_stride];
+                y_now[t] = y_in[t * args.y_stride];
             }
         float product = 1.0f, end = 0.0f;
 #pragma unroll
         for (int t = 0; t < UNIT_RUN; ++t) {
             a[t] = 1.0f;                          // tokens past the end keep the state as it is
             b[t] = 0.0f;
-            if (live && t0 + t < count) unit_terms<T>(pre_r[t], pre_i[t], to_float<T>(u_now[t]), br, bi, c, a[t], b[t]);
+            if (t < here) unit_terms<T>(pre_r[t], pre_i[t], to_float<T>(u_now[t]), br, bi, c, a[t], b[t]);
             product = __fmul_rn(product, a[t]);
             end = __fmaf_rn(a[t], end, b[t]);
         }
         products[turn][warp][lane] = product;
         ends[turn][warp][lane] = end;
-        __syncthreads();                          // also: the carry of the block before is there
-        float s = carry[turn ^ 1][lane];
+        __syncthreads();
+        if (ctas > 1) {
+            if (warp == 0) {                      // the CTA's tokens as one, for the other CTAs
+                float all = 1.0f, s = 0.0f;
+#pragma unroll
+                for (int w = 0; w < UNIT_WARPS; ++w) {
+                    s = __fmaf_rn(products[turn][w][lane], s, ends[turn][w][lane]);
+                    all = __fmul_rn(all, products[turn][w][lane]);
+                }
+                block_product[turn][lane] = all;
+                block_end[turn][lane] = s;
+            }
+            cluster_arrive();
+            cluster_wait();
+        }
+        float s = carry;
+        if (ctas > 1) {
+            for (int r = 0; r < ctas; ++r) {      // to this CTA's tokens, and on to the next round's
+                if (r == rank) s = carry;
+                carry = __fmaf_rn(load_of_cta(&block_product[turn][lane], r), carry, load_of_cta(&block_end[turn][lane], r));
+            }
+        } else {
+#pragma unroll
+            for (int w = 0; w < UNIT_WARPS; ++w) carry = __fmaf_rn(products[turn][w][lane], carry, ends[turn][w][lane]);
+        }
         for (int w = 0; w < warp; ++w) s = __fmaf_rn(products[turn][w][lane], s, ends[turn][w][lane]);
 #pragma unroll
         for (int t = 0; t < UNIT_RUN; ++t) {
             s = __fmaf_rn(a[t], s, b[t]);
-            if (live && t0 + t < count)
-                dst[(int64_t)(t0 + t) * args.out_stride] =
+            if (t < here)
+                dst[t * args.out_stride] =
                     from_float<T>(__fmul_rn(s, branch_act<T>(__fadd_rn(to_float<T>(y_now[t]), by), args.act)));
         }
-        if (warp == UNIT_WARPS - 1) {
-            carry[turn][lane] = s;
-            if (first + UNIT_BLOCK >= count && live) mine[0] = s;
-        }
+        t0 += step;
+        u_in += (int64_t)step * args.u_stride;
+        y_in += (int64_t)step * args.y_stride;
+        dst += (int64_t)step * args.out_stride;
+        pre_in += (int64_t)step * args.pre_token;
+    }
+    if (rank == 0 && warp == 0 && live) mine[0] = carry;
+    if (ctas > 1) {                               // no CTA leaves while another reads its shared memory
+        cluster_arrive();
+        cluster_wait();
     }
 }
 
@@ -161,10 +205,28 @@ __global__ void __launch_bounds__(128) recurrent_unit_step_kernel(const T* __res
 // One token a request, the gates' products inside.  A CTA takes GATE_CHANNELS channels of one block of gates for up to
 // ROWS requests: u of the block waits in shared memory (float32), a warp takes a channel at a time, its lanes eight (or
 // one) neighbouring weights of the channel's two rows, and the 2 ROWS sums are added by halving over the lanes.
-#define GATE_CHANNELS 16
+#define GATE_CHANNELS 8
 #define GATE_WARPS 4
-__device__ __forceinline__ void load_many(const float* p, float* v) { load_values<4>(p, v); load_values<4>(p + 4, v + 4); }
-__device__ __forceinline__ void load_many(const bf16* p, float* v) { unpack_bf16x8(*reinterpret_cast<const uint4*>(p), v); }
+// VEC neighbouring weights as they were loaded
+template <typename T, int VEC> struct Weights;
+template <typename T> struct Weights<T, 1> {
+    T v;
+    __device__ __forceinline__ void load(const T* p) { v = *p; }
+    __device__ __forceinline__ void spread(float* x) const { x[0] = to_float<T>(v); }
+};
+template <> struct Weights<float, 8> {
+    float v[8];
+    __device__ __forceinline__ void load(const float* p) { load_values<4>(p, v); load_values<4>(p + 4, v + 4); }
+    __device__ __forceinline__ void spread(float* x) const {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] = v[i];
+    }
+};
+template <> struct Weights<bf16, 8> {
+    uint4 v;
+    __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void spread(float* x) const { unpack_bf16x8(v, x); }
+};
 
 template <typename T, int ROWS, int VEC>
 __global__ void __launch_bounds__(GATE_WARPS * 32) recurrent_unit_gated_step_kernel(
@@ -177,21 +239,35 @@ __global__ void __launch_bounds__(GATE_WARPS * 32) recurrent_unit_gated_step_ker
     const int block = blockIdx.x / parts, j0 = blockIdx.x % parts * GATE_CHANNELS;
     const int row0 = blockIdx.y * ROWS, here = min(ROWS, rows - row0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    constexpr int MINE = GATE_CHANNELS / GATE_WARPS;                  // a warp's channels: their first weights are on
+    Weights<T, VEC> ahead_r[MINE], ahead_i[MINE];                    // their way before u is there
+#pragma unroll
+    for (int i = 0; i < MINE; ++i) {
+        const int j = j0 + warp + i * GATE_WARPS;
+        if (j < size && lane * VEC < size) {
+            const T* w_r = w + ((int64_t)block * 2 * size + j) * size + lane * VEC;
+            ahead_r[i].load(w_r);
+            ahead_i[i].load(w_r + (int64_t)size * size);
+        }
+    }
     for (int e = threadIdx.x; e < ROWS * padded; e += GATE_WARPS * 32) {
         const int q = e / padded, k = e % padded;
         u_s[e] = q < here && k < size ? to_float<T>(u[(int64_t)args.row_starts[row0 + q] * args.u_stride + block * size + k]) : 0.0f;
     }
     __syncthreads();
-    for (int c = warp; c < GATE_CHANNELS && j0 + c < size; c += GATE_WARPS) {
+#pragma unroll
+    for (int i = 0; i < MINE; ++i) {
+        const int c = warp + i * GATE_WARPS;
+        if (j0 + c >= size) break;
         const T* w_r = w + ((int64_t)block * 2 * size + j0 + c) * size;
         const T* w_i = w_r + (int64_t)size * size;
         float sums[SUMS];
 #pragma unroll
-        for (int i = 0; i < SUMS; ++i) sums[i] = 0.0f;
+        for (int e = 0; e < SUMS; ++e) sums[e] = 0.0f;
         for (int k = lane * VEC; k < size; k += 32 * VEC) {
             float r[VEC], in[VEC];
-            if constexpr (VEC == 8) { load_many(w_r + k, r); load_many(w_i + k, in); }
-            else { r[0] = to_float<T>(w_r[k]); in[0] = to_float<T>(w_i[k]); }
+            if (k == lane * VEC) { ahead_r[i].spread(r); ahead_i[i].spread(in); }
+            else { Weights<T, VEC> x; x.load(w_r + k); x.spread(r); x.load(w_i + k); x.spread(in); }
 #pragma unroll
             for (int q = 0; q < ROWS; ++q) {
                 float x[VEC];
@@ -211,9 +287,9 @@ __global__ void __launch_bounds__(GATE_WARPS * 32) recurrent_unit_gated_step_ker
             if (n > 1) {
                 const bool upper = (lane & bit) != 0;
 #pragma unroll
-                for (int i = 0; i < n / 2; ++i) {
-                    const float hand = upper ? sums[i] : sums[i + n / 2], keep = upper ? sums[i + n / 2] : sums[i];
-                    sums[i] = keep + __shfl_xor_sync(0xffffffffu, hand, bit);
+                for (int e = 0; e < n / 2; ++e) {
+                    const float hand = upper ? sums[e] : sums[e + n / 2], keep = upper ? sums[e + n / 2] : sums[e];
+                    sums[e] = keep + __shfl_xor_sync(0xffffffffu, hand, bit);
                 }
                 if (upper) owner += n / 2;
                 n >>= 1;
@@ -245,13 +321,14 @@ __global__ void __launch_bounds__(GATE_WARPS * 32) recurrent_unit_gated_step_ker
 // u, y, out: [tokens, >= channels] of the storage type with row strides; pre float32 with strides for the token and for
 // the block of gates (`size` channels each; r's pre-activations, then i's), or, with `single`, null and w [blocks, 2
 // size, size] of the storage type (u's products are done here); bias_r, bias_i, decay float32 [channels], bias_y too
-// or null; state float32 [slots, channels].  `single`: every entry is one token.
+// or null; state float32 [slots, channels].  `single`: every entry is one token; `tokens`: of all
+// entries.
 extern "C" int tvb_recurrent_unit(const void* u, long long u_stride, const void* y, long long y_stride, const float* pre,
                                   long long pre_token, long long pre_block, const void* w, const float* bias_r,
                                   const float* bias_i, const float* decay, const float* bias_y, float* state,
                                   const int* row_starts, const int* state_slots, const int* token_row, void* out,
-                                  long long out_stride, int rows, int channels, int size, int act, int single, int dtype,
-                                  void* stream) {
+                                  long long out_stride, int rows, int tokens, int channels, int size, int act, int single,
+                                  int dtype, void* stream) {
     if (rows <= 0) return 0;
     if (channels <= 0 || size <= 0 || channels % size || rows > 65535 || act < 0 || act > 2 || !state || !bias_r || !bias_i ||
         !decay || (!pre == !w) || (w && !single))
@@ -291,11 +368,17 @@ extern "C" int tvb_recurrent_unit(const void* u, long long u_stride, const void*
         else return TVB_BAD_ARGUMENT;
         return tvb_last_error();
     }
-    const dim3 grid((channels + 31) / 32, rows);
+    // as many CTAs a cluster as the step's longest entry could use, while SMs would idle otherwise
+    const int groups = (channels + 31) / 32;
+    int ctas = 1;
+    while (ctas < UNIT_MOST_CTAS && 2 * ctas * UNIT_BLOCK <= tokens && (long long)groups * rows * ctas < 4 * 148) ctas *= 2;
+    if (groups > 65535) return TVB_BAD_ARGUMENT;
+    TvbLaunch launch(dim3(ctas, groups, rows), dim3(UNIT_WARPS * 32), 0, s, 0, ctas);
+    cudaError_t e;
     if (dtype == TVB_F32)
-        recurrent_unit_scan_kernel<float><<<grid, UNIT_WARPS * 32, 0, s>>>((const float*)u, (const float*)y, (float*)out, args);
+        e = cudaLaunchKernelEx(&launch.config, recurrent_unit_scan_kernel<float>, (const float*)u, (const float*)y, (float*)out, args, ctas);
     else if (dtype == TVB_BF16)
-        recurrent_unit_scan_kernel<bf16><<<grid, UNIT_WARPS * 32, 0, s>>>((const bf16*)u, (const bf16*)y, (bf16*)out, args);
+        e = cudaLaunchKernelEx(&launch.config, recurrent_unit_scan_kernel<bf16>, (const bf16*)u, (const bf16*)y, (bf16*)out, args, ctas);
     else return TVB_BAD_ARGUMENT;
-    return tvb_last_error();
+    return e == cudaSuccess ? tvb_last_error() : (int)e;
 }

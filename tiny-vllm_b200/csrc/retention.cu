@@ -631,30 +631,66 @@ extern "C" int tvb_gated_step(const void* proj, long long token_stride, int q_at
 }
 
 // A warp a (token, head): o / sqrt(mean(o^2) + eps) (with `unit_norm`; times `norm_weight` [vdim], one for all
-// heads, if given), times act(gate).
-template <typename T>
+// heads, if given), times act(gate).  VEC: neighbouring values a lane moves at once, 4 or 1; up to FINISH_HELD times as
+// many wait in registers between the sum of squares and the result.
+#define FINISH_HELD 2
+template <typename T, int VEC>
 __global__ void __launch_bounds__(128) retention_finish_kernel(
-    const float* __restrict__ o, const T* gate, int64_t gate_stride, T* __restrict__ out, int64_t out_stride,
+    const float* __restrict__ o, const T* __restrict__ gate, int64_t gate_stride, T* __restrict__ out, int64_t out_stride,
     int tokens, int heads, int vdim, int unit_norm, float eps, int act, const float* __restrict__ norm_weight) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t item = (int64_t)blockIdx.x * 4 + warp;
     if (item >= (int64_t)tokens * heads) return;
     const int token = (int)(item / heads), head = (int)(item % heads);
     const float* src = o + ((int64_t)token * heads + head) * vdim;
+    const T* g = gate ? gate + (int64_t)token * gate_stride + (int64_t)head * vdim : nullptr;
+    T* dst = out + (int64_t)token * out_stride + (int64_t)head * vdim;
+    float held[FINISH_HELD][VEC], z[FINISH_HELD][VEC];
+#pragma unroll
+    for (int j = 0; j < FINISH_HELD; ++j) {
+        const int i = (lane + 32 * j) * VEC;
+        if (i < vdim) {
+            load_values<VEC>(src + i, held[j]);
+            if (g) load_values<VEC>(g + i, z[j]);
+        }
+    }
     float factor = 1.0f;
     if (unit_norm) {
         float squares = 0.0f;
-        for (int i = lane; i < vdim; i += 32) squares = __fmaf_rn(src[i], src[i], squares);
+#pragma unroll
+        for (int j = 0; j < FINISH_HELD; ++j)
+            if ((lane + 32 * j) * VEC < vdim) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) squares = __fmaf_rn(held[j][e], held[j][e], squares);
+            }
+        for (int i = (lane + 32 * FINISH_HELD) * VEC; i < vdim; i += 32 * VEC) {
+            float x[VEC];
+            load_values<VEC>(src + i, x);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) squares = __fmaf_rn(x[e], x[e], squares);
+        }
         squares = warp_sum(squares);
         factor = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(squares, (float)vdim), eps)));
     }
-    const T* g = gate ? gate + (int64_t)token * gate_stride + (int64_t)head * vdim : nullptr;
-    T* dst = out + (int64_t)token * out_stride + (int64_t)head * vdim;
-    for (int i = lane; i < vdim; i += 32) {
-        float x = __fmul_rn(src[i], factor);
-        if (norm_weight) x = __fmul_rn(x, norm_weight[i]);
-        if (g) x = __fmul_rn(x, output_gate(to_float<T>(g[i]), act));
-        dst[i] = from_float<T>(x);
+    auto finish = [&](float* x, const float* gates, int i) {
+        float weight[VEC];
+        if (norm_weight) load_values<VEC>(norm_weight + i, weight);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            x[e] = __fmul_rn(x[e], factor);
+            if (norm_weight) x[e] = __fmul_rn(x[e], weight[e]);
+            if (g) x[e] = __fmul_rn(x[e], act == RET_ACT_SILU ? silu_for<T>(gates[e]) : output_gate(gates[e], act));
+        }
+        store_values<VEC>(dst + i, x);
+    };
+#pragma unroll
+    for (int j = 0; j < FINISH_HELD; ++j)
+        if ((lane + 32 * j) * VEC < vdim) finish(held[j], z[j], (lane + 32 * j) * VEC);
+    for (int i = (lane + 32 * FINISH_HELD) * VEC; i < vdim; i += 32 * VEC) {
+        float x[VEC], gates[VEC];
+        load_values<VEC>(src + i, x);
+        if (g) load_values<VEC>(g + i, gates);
+        finish(x, gates, i);
     }
 }
 
@@ -769,12 +805,14 @@ extern "C" int tvb_retention_finish(const float* o, const void* gate, long long 
     const long long blocks = ((long long)tokens * heads + 3) / 4;
     if (blocks > 2147483647LL) return TVB_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == TVB_F32)
-        retention_finish_kernel<float><<<(unsigned)blocks, 128, 0, s>>>(o, (const float*)gate, gate_stride, (float*)out,
-                                                                        out_stride, tokens, heads, vdim, unit_norm, eps, act, norm_weight);
-    else if (dtype == TVB_BF16)
-        retention_finish_kernel<bf16><<<(unsigned)blocks, 128, 0, s>>>(o, (const bf16*)gate, gate_stride, (bf16*)out,
-                                                                       out_stride, tokens, heads, vdim, unit_norm, eps, act, norm_weight);
+    const size_t element = dtype == TVB_BF16 ? 2 : 4;
+    const bool by_four = vdim % 4 == 0 && out_stride % 4 == 0 && (!gate || gate_stride % 4 == 0) &&
+                         ((uintptr_t)o | (uintptr_t)norm_weight) % 16 == 0 && ((uintptr_t)gate | (uintptr_t)out) % (4 * element) == 0;
+#define GO(T, VEC) retention_finish_kernel<T, VEC><<<(unsigned)blocks, 128, 0, s>>>(                                   \
+        o, (const T*)gate, gate_stride, (T*)out, out_stride, tokens, heads, vdim, unit_norm, eps, act, norm_weight)
+    if (dtype == TVB_F32) { if (by_four) GO(float, 4); else GO(float, 1); }
+    else if (dtype == TVB_BF16) { if (by_four) GO(bf16, 4); else GO(bf16, 1); }
     else return TVB_BAD_ARGUMENT;
+#undef GO
     return tvb_last_error();
 }

@@ -1168,15 +1168,21 @@ def selective_scan(x: torch.Tensor, *, pre: torch.Tensor | None, z: torch.Tensor
 
 # ------------------------------------- linear recurrent unit: a number of state a channel, gates from square matrices
 UNIT_ACTS = {None: 0, "silu": 1, "gelu_tanh": 2}
-UNIT_STEP_ROWS = 16               # requests up to which the step kernel does the gates' products itself
+UNIT_STEP_ROWS = 4                # requests up to which the step kernel does the gates' products itself
 UNIT_STEP_FLOATS = 40 * 1024 // 4  # float32 numbers of u that wait in its shared memory
 
 
-def recurrent_unit_step_takes(rows: int, size: int) -> bool:
-    """Whether a step of single tokens does the gates' products (square matrices of ``size``) inside the step kernel:
-    its CTAs read the weights once for up to eight requests."""
+def _unit_step_fits(rows: int, size: int) -> bool:
+    """Whether u of one block of gates waits in the step kernel's shared memory (for up to eight requests at a time)."""
     together = 1 if rows <= 1 else 2 if rows == 2 else 4 if rows <= 4 else 8
-    return rows <= UNIT_STEP_ROWS and together * (-(-size // 8) * 8) <= UNIT_STEP_FLOATS
+    return together * (-(-size // 8) * 8) <= UNIT_STEP_FLOATS
+
+
+def recurrent_unit_step_takes(rows: int, size: int) -> bool:
+    """Whether a step of single tokens does the gates' products (square matrices of ``size``) inside the step kernel.
+    For few requests that is cheaper than a launch of its own (us, one launch / two and what lies between them: one
+    request of 4,096 channels in 32 blocks 3.6 / 5.0, of 1,024 in 16 3.3 / 4.7; eight requests 6.8 / 5.1 and 4.9 / 4.8)."""
+    return rows <= UNIT_STEP_ROWS and _unit_step_fits(rows, size)
 
 
 def block_products(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -1238,23 +1244,24 @@ def recurrent_unit(u: torch.Tensor, y: torch.Tensor, *, blocks: int, decay: torc
     if pre is not None and (pre.dtype != torch.float32 or pre.shape != (tokens, blocks, 2 * size) or pre.stride(2) != 1):
         raise KernelError("recurrent_unit: pre must be float32 [tokens, blocks, 2 * size]")
     if weight is not None and (weight.dtype != u.dtype or weight.shape != (blocks, 2 * size, size)
-                               or not weight.is_contiguous() or not recurrent_unit_step_takes(min(rows, UNIT_STEP_ROWS), size)):
+                               or not weight.is_contiguous() or not _unit_step_fits(rows, size)):
         raise KernelError("recurrent_unit: weight must be contiguous [blocks, 2 * size, size] of the dtype of u, of a "
                           "size that waits in shared memory")
     fn = _fn("recurrent_unit", "tvb_recurrent_unit",
              [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p,
               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
-              c_int, c_int, c_void_p])
+              c_int, c_int, c_int, c_void_p])
     _check(fn(u.data_ptr(), u.stride(0), y.data_ptr(), y.stride(0), _ptr(pre), 0 if pre is None else pre.stride(0),
               0 if pre is None else pre.stride(1), _ptr(weight), bias_r.data_ptr(), bias_i.data_ptr(), decay.data_ptr(),
               _ptr(bias_y), state.data_ptr(), row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(),
-              out.data_ptr(), out.stride(0), rows, channels, size, UNIT_ACTS[act], 1 if single else 0, dtype_tag(u.dtype),
-              _stream()), "recurrent_unit")
+              out.data_ptr(), out.stride(0), rows, tokens, channels, size, UNIT_ACTS[act], 1 if single else 0,
+              dtype_tag(u.dtype), _stream()), "recurrent_unit")
     return out
 
 
 # ------------------------------------------------------------------------------------- gated delta rule
 DELTA_MAX_DIM = 256
+DELTA_BLOCK, DELTA_COEFFICIENTS = 8, 152     # tokens a piece of the scan, numbers that say how they act on one another
 DELTA_MAX_STEP_GROUPS = 256       # columns (in fours, where they fit) of a head that the step kernel takes
 
 
@@ -1272,7 +1279,7 @@ def delta_rule(mixed: torch.Tensor, proj: torch.Tensor, *, q_at: int, k_at: int,
                query_scale: float = 1.0, unit_eps: float = 1e-6, unit_norm: bool = True,
                norm_weight: torch.Tensor | None = None, eps: float = 0.0, gate_at: int | None = None,
                gate_act: str | None = "silu", out: torch.Tensor | None = None,
-               raw_out: torch.Tensor | None = None) -> torch.Tensor:
+               raw_out: torch.Tensor | None = None, cols: int = 0) -> torch.Tensor:
     """The gated delta rule between a mixer's convolution and its output projection.
 
     ``mixed`` [tokens, columns] (convolved) holds q heads (``key_heads`` of ``dim``) from ``q_at``, k heads from ``k_at``
@@ -1286,7 +1293,7 @@ def delta_rule(mixed: torch.Tensor, proj: torch.Tensor, *, q_at: int, k_at: int,
     [vdim]) and act(gate), and rounded to the storage type: [tokens, heads * vdim].  ``raw_out`` (float32) receives o.
 
     A step in which every entry is one token runs as one launch, a CTA a (request, head), unless ``raw_out`` asks for the
-    scan."""
+    scan, whose threads hold ``cols`` (2 or 4; 0: chosen) value columns."""
     _need_cuda(mixed, proj, rate, dt_bias, norm_weight, state, row_starts, state_slots, token_row, out, raw_out)
     tokens = mixed.shape[0]
     rows = _entry_checks("delta_rule", tokens, row_starts, state_slots, token_row)
@@ -1330,19 +1337,21 @@ def delta_rule(mixed: torch.Tensor, proj: torch.Tensor, *, q_at: int, k_at: int,
         raise KernelError("delta_rule: raw_out must be contiguous float32 [tokens, heads * vdim]")
     padded = -(-dim // 4) * 4
     vectors = torch.empty((2, tokens, key_heads, padded), dtype=torch.float32, device=mixed.device)
-    scalars = torch.empty((tokens, heads, 4), dtype=torch.float32, device=mixed.device)
+    pieces = tokens // DELTA_BLOCK + rows
+    coefficients = torch.empty((pieces, heads, DELTA_COEFFICIENTS), dtype=torch.float32, device=mixed.device)
     fn = _fn("delta_rule", "tvb_delta_prepare",
              [c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
-              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(mixed.data_ptr(), mixed.stride(0), q_at, k_at, proj.data_ptr(), proj.stride(0), beta_at, decay_at,
               rate.data_ptr(), dt_bias.data_ptr(), query_scale, unit_eps, vectors[0].data_ptr(), vectors[1].data_ptr(),
-              scalars.data_ptr(), tokens, key_heads, group, dim, padded, tag, _stream()), "delta_prepare")
+              coefficients.data_ptr(), row_starts.data_ptr(), token_row.data_ptr(), rows, pieces, key_heads, group, dim,
+              padded, tag, _stream()), "delta_prepare")
     fn = _fn("delta_rule", "tvb_delta_scan",
              [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-              c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(vectors[0].data_ptr(), vectors[1].data_ptr(), scalars.data_ptr(), mixed.data_ptr() + v_at * element,
+              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(vectors[0].data_ptr(), vectors[1].data_ptr(), coefficients.data_ptr(), mixed.data_ptr() + v_at * element,
               mixed.stride(0), state.data_ptr(), row_starts.data_ptr(), state_slots.data_ptr(), token_row.data_ptr(),
-              raw_out.data_ptr(), rows, heads, group, dim, padded, vdim, tag, _stream()), "delta_scan")
+              raw_out.data_ptr(), rows, heads, group, dim, padded, vdim, cols, tag, _stream()), "delta_scan")
     finish = _fn_of("retention", "tvb_retention_finish", _RETENTION_FINISH_ARGS)
     gate_ptr = None if gate_at is None else proj.data_ptr() + gate_at * element
     _check(finish(raw_out.data_ptr(), gate_ptr, proj.stride(0), out.data_ptr(), out.stride(0), tokens, heads, vdim,
