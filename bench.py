@@ -1736,7 +1736,10 @@ def lasupel_roofline(name: str, size: str, tokens: int, context: int, peak: dict
     elif name == "short_convolution":                                 # of the unit and of the delta rule in turn
         bytes_ = tokens * (width + 2 * heads * dim) / 2 * (2 * 2 + (0 if prompt else (LASUPEL_TAPS - 1) * 4 * 2))
     elif name == "recurrent_unit":
-        bytes_ = tokens * width * (2 + 2 + 2 + (8 if prompt else 4 * 2)) + (0 if prompt else 2 * width * part * 2)
+        # u, y, the result and the gates' pre-activations (few requests: the gates' weights instead), the state twice
+        from tinyvllm_b200.ops import kernels
+        inside = not prompt and kernels.recurrent_unit_step_takes(tokens, part)
+        bytes_ = tokens * width * (2 + 2 + 2 + (0 if inside else 8) + (0 if prompt else 8)) + (2 * width * part * 2 if inside else 0)
     elif name == "block_products":
         bytes_ = tokens * width * (2 + 8) + 2 * width * part * 2
         limits.append((2.0 * tokens * width * 2 * part / (peak["bf16_tflops"] * 1e12), "tensor"))
